@@ -123,6 +123,14 @@ class StreamMixSpec:
 
 
 @dataclass(frozen=True)
+class StreamJoinSpec:
+    """What the stream becomes before a call whose `join` is set: a product of the stream and the embedding's output."""
+    kind: str                    # key in parts.STREAM_JOINS
+    width: int
+    options: tuple = ()
+
+
+@dataclass(frozen=True)
 class LayerSpec:
     """One block: `arrangement` names how the parts are wired (parts.ARRANGEMENTS); `parts` holds one spec record
     for each part name the arrangement declares (its PARTS), as (name, spec) pairs.  `LayerSpec.of("prenorm",
@@ -177,11 +185,13 @@ class LayerCall:
     state:  index of a second cache entry, of kind "state", that the call's mixer keeps beside the first
             (what a short convolution remembers of a request's last tokens, say); None if it keeps none.
             The mixer's class names its shape with `state_need(spec)`.
+    join:   whether the model's stream join (ModelSpec.join) replaces the stream right before this call.
     """
     layer: int
     cache: int
     write: bool = True
     state: int | None = None
+    join: bool = False
 
 
 @dataclass(frozen=True)
@@ -198,6 +208,7 @@ class ModelSpec:
     logit_scale: float = 1.0
     embedding: EmbeddingSpec | None = None     # None: a plain table of [vocab, width] scaled by embedding_scale
     head: HeadSpec | None = None               # None: a plain [vocab, width] projection scaled by logit_scale
+    join: StreamJoinSpec | None = None         # what the calls marked `join` enter through
 
     def embedding_spec(self) -> EmbeddingSpec:
         return self.embedding or EmbeddingSpec("table", self.vocab, self.width, self.embedding_scale)

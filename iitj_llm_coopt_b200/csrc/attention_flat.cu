@@ -5,7 +5,8 @@
 //
 // llm_latent_prepare:  per token, from the fused projection row [heads x (dim + rot_dim) | kv_rank | rot_dim]:
 //                      latent = rmsnorm(row[kv_rank part]) * gain, shared key part rotated, both stored as one cache row;
-//                      every head's rotated query part written behind the place of its absorbed part in q_out.
+//                      every head's rotated query part written behind the place of its absorbed part in q_out.  A gate's number
+//                      per head that follows in the row is copied out as float32 on request.
 // llm_headnorm_store:  per token, every query head and key head divided by its root mean square and multiplied by a
 //                      gain vector shared by all heads (optional); queries in place, keys and values into the cache.
 // llm_attention_flat:  softmax(score) over the keys [max(0, p - window + 1), p] (window 0: from 0), times the values,
@@ -41,20 +42,34 @@ __global__ void __launch_bounds__(128)
 latent_prepare_kernel(const T* __restrict__ qd, int ld, const T* __restrict__ kv, int ld_kv, const float* __restrict__ cos,
                       const float* __restrict__ sin, int rotary_dim,
                       int interleaved, const float* __restrict__ gain, float eps, T* __restrict__ q_out, T* __restrict__ cache,
-                      const int* __restrict__ slots, long long page_stride, int page_size, int heads, int dim, int rot_dim, int rank) {
+                      const int* __restrict__ slots, long long page_stride, int page_size, int heads, int dim, int rot_dim, int rank,
+                      float* __restrict__ gate_out) {
     pdl_trigger();
     pdl_wait();
     __shared__ float red[32];
     const int t = blockIdx.x;
     const T* row = qd + (size_t)t * ld;
     const T* low = kv + (size_t)t * ld_kv;             // [rank latent numbers | rot_dim numbers of the shared key part]
-    const int out_row = rank + rot_dim;
-    const float* cos_t = cos ? cos + (size_t)t * (rotary_dim / 2) : nullptr;
-    const float* sin_t = sin ? sin + (size_t)t * (rotary_dim / 2) : nullptr;
-    // every head's rotated query part
-    for (int h = 0; h < heads; ++h)
-        rotate_row(row + h * (dim + rot_dim) + dim, q_out + (size_t)t * heads * out_row + (size_t)h * out_row + rank, rot_dim,
-                   rotary_dim, interleaved, cos_t, sin_t, threadIdx.x, blockDim.x);
+    const int out_row = rank + rot_dim, half = rotary_dim / 2;
+    const float* cos_t = cos ? cos + (size_t)t * half : nullptr;
+    const float* sin_t = sin ? sin + (size_t)t * half : nullptr;
+    // every head's rotated query part: the pairs of all heads one after the other, then what is not rotated
+    for (int w = threadIdx.x; w < heads * half; w += blockDim.x) {
+        const int h = w / half, p = w - h * half;
+        const T* in = row + (size_t)h * (dim + rot_dim) + dim;
+        T* to = q_out + (size_t)t * heads * out_row + (size_t)h * out_row + rank;
+        const int a = interleaved ? 2 * p : p, b = interleaved ? 2 * p + 1 : p + half;
+        const float x = to_f32(in[a]), y = to_f32(in[b]), c = cos_t[p], s = sin_t[p];
+        to[a] = from_f32<T>(x * c - y * s);
+        to[b] = from_f32<T>(y * c + x * s);
+    }
+    const int rest = rot_dim - rotary_dim;
+    for (int w = threadIdx.x; w < heads * rest; w += blockDim.x) {
+        const int h = w / rest, i = rotary_dim + (w - h * rest);
+        q_out[(size_t)t * heads * out_row + (size_t)h * out_row + rank + i] = row[(size_t)h * (dim + rot_dim) + dim + i];
+    }
+    if (gate_out)
+        for (int h = threadIdx.x; h < heads; h += blockDim.x) gate_out[(size_t)t * heads + h] = to_f32(low[out_row + h]);
     // the latent row's statistics (all threads take part, whether the row is stored or not)
     float ss = 0.f;
     for (int i = threadIdx.x; i < rank; i += blockDim.x) {
@@ -227,14 +242,16 @@ attention_flat_kernel(const T* __restrict__ q, int q_stride, const T* __restrict
 LLM_API int llm_latent_prepare(const void* qd, int ld, const void* kv, int ld_kv, const float* cos, const float* sin,
                                int rotary_dim, int interleaved,
                                const float* gain, float eps, void* q_out, void* cache, const int* slots, long long page_stride,
-                               int page_size, int dtype, int tokens, int heads, int dim, int rot_dim, int rank, cudaStream_t stream) {
+                               int page_size, int dtype, int tokens, int heads, int dim, int rot_dim, int rank, float* gate_out,
+                               cudaStream_t stream) {
     if (tokens == 0) return 0;
     if (rotary_dim % 2 || rotary_dim > rot_dim || (rotary_dim && (!cos || !sin)))
         LLM_FAIL(-1, "latent_prepare: rotary_dim %d must be even, at most rot_dim %d, and come with tables", rotary_dim, rot_dim);
     return llm_dispatch_dtype(dtype, [&](auto tag) {
         using T = decltype(tag);
         llm_launch(latent_prepare_kernel<T>, (unsigned)tokens, 128, 0, stream, (const T*)qd, ld, (const T*)kv, ld_kv, cos, sin,
-                   rotary_dim, interleaved, gain, eps, (T*)q_out, (T*)cache, slots, page_stride, page_size, heads, dim, rot_dim, rank);
+                   rotary_dim, interleaved, gain, eps, (T*)q_out, (T*)cache, slots, page_stride, page_size, heads, dim, rot_dim, rank,
+                   gate_out);
         LLM_CHECK_LAUNCH("latent_prepare");
         return 0;
     });

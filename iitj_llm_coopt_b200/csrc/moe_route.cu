@@ -4,7 +4,9 @@
 // llm_route_topk:   s = softmax(z) over all router outputs, or sigmoid(z) of each (float32); the `top` largest of
 //                   s + correction (null: of s) are chosen (ties: the lower index), in descending order; the weights are the
 //                   chosen s, not renormalised.  A third form compares z + bias itself (the bias where `correction` would be) and
-//                   takes the softmax over the chosen outputs alone as weights.  One warp per token.
+//                   takes the softmax over the chosen outputs alone as weights.  With `groups` > 1 the outputs form that many
+//                   equal groups of neighbours and only those of the `keep` groups with the largest single entry can be chosen
+//                   (ties: the lower group).  With `tiny` > 0 the weights are divided by (their sum + tiny).  One warp per token.
 // llm_moe_plan:     the (token, choice) pairs sorted by expert, stable in the pair's index: source[r] = token of sorted row r,
 //                   place[token * top + j] = sorted row of that pair (-1 for a choice >= experts: an expert without tensors),
 //                   and the list of row tiles (expert, first row, rows) that llm_gemm_grouped walks, with its count in front.
@@ -17,14 +19,14 @@ namespace {
 
 __global__ void __launch_bounds__(128)
 route_topk_kernel(const float* __restrict__ z, const float* __restrict__ correction, int* __restrict__ chosen,
-                  float* __restrict__ weights, int tokens, int outputs, int top, int sigmoid) {
+                  float* __restrict__ weights, int tokens, int outputs, int top, int sigmoid, int groups, int keep, float tiny) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float route_smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * (blockDim.x >> 5) + warp;
     if (t >= tokens) return;
-    float* s = route_smem + (size_t)warp * 2 * outputs;      // scores, then choice scores
+    float* s = route_smem + (size_t)warp * (2 * outputs + groups);      // scores, then choice scores, then the groups' worth
     float* c = s + outputs;
     const float* row = z + (size_t)t * outputs;
     if (sigmoid == 2) {
@@ -43,6 +45,25 @@ route_topk_kernel(const float* __restrict__ z, const float* __restrict__ correct
         for (int i = lane; i < outputs; i += 32) { s[i] *= inv; c[i] = s[i] + (correction ? correction[i] : 0.f); }
     }
     __syncwarp();
+    if (keep < groups) {
+        // a group is worth its largest entry; a closed group's entries drop out of the choice
+        float* worth = c + outputs;
+        const int size = outputs / groups;
+        for (int g = lane; g < groups; g += 32) {
+            float m = -INFINITY;
+            for (int i = 0; i < size; ++i) m = fmaxf(m, c[g * size + i]);
+            worth[g] = m;
+        }
+        __syncwarp();
+        for (int g = lane; g < groups; g += 32) {
+            int better = 0;
+            for (int o = 0; o < groups; ++o) better += worth[o] > worth[g] || (worth[o] == worth[g] && o < g);
+            if (better >= keep)
+                for (int i = 0; i < size; ++i) c[g * size + i] = -INFINITY;
+        }
+        __syncwarp();
+    }
+    float total = 0.f;
     for (int j = 0; j < top; ++j) {
         float best = -INFINITY;
         int at = 0x7fffffff;
@@ -54,6 +75,8 @@ route_topk_kernel(const float* __restrict__ z, const float* __restrict__ correct
             const int oa = __shfl_xor_sync(0xffffffffu, at, o);
             if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
         }
+        if (at >= outputs) at = 0;                          // nothing compares (the scores are no numbers): stay in range
+        total += s[at];
         if (lane == 0) {
             chosen[(size_t)t * top + j] = at;
             weights[(size_t)t * top + j] = s[at];
@@ -61,6 +84,8 @@ route_topk_kernel(const float* __restrict__ z, const float* __restrict__ correct
         }
         __syncwarp();
     }
+    if (tiny > 0.f && lane == 0)
+        for (int j = 0; j < top; ++j) weights[(size_t)t * top + j] /= total + tiny;
     if (sigmoid == 2 && lane == 0) {
         // softmax over the chosen outputs alone; the first choice is the largest
         float* w = weights + (size_t)t * top;
@@ -191,14 +216,18 @@ LLM_API int llm_gather_rows(const void* src, const int* index, const int* live_r
 }
 
 LLM_API int llm_route_topk(const float* z, const float* correction, int* chosen, float* weights, int tokens, int outputs, int top,
-                           int sigmoid, cudaStream_t stream) {
+                           int sigmoid, int groups, int keep, float tiny, cudaStream_t stream) {
     if (tokens == 0) return 0;
     if (top < 1 || top > outputs) LLM_FAIL(-1, "route_topk: %d of %d outputs", top, outputs);
     if (sigmoid < 0 || sigmoid > 2) LLM_FAIL(-1, "route_topk: form %d is not known (0 softmax, 1 sigmoid, 2 softmax over the chosen)", sigmoid);
-    const size_t smem = (size_t)4 * 2 * outputs * sizeof(float);
-    if (smem > 48 * 1024) LLM_FAIL(-1, "route_topk: %d router outputs are more than 1536", outputs);
+    if (groups < 1 || outputs % groups || keep < 1 || keep > groups || top > outputs / groups * keep)
+        LLM_FAIL(-1, "route_topk: %d of %d outputs from %d of %d equal groups", top, outputs, keep, groups);
+    if (tiny > 0.f && sigmoid == 2) LLM_FAIL(-1, "route_topk: the softmax over the chosen sums to one already");
+    if (keep == groups) groups = keep = 0;                  // every group is open
+    const size_t smem = (size_t)4 * (2 * outputs + groups) * sizeof(float);
+    if (smem > 48 * 1024) LLM_FAIL(-1, "route_topk: %d router outputs in %d groups are too many for a block", outputs, groups);
     llm_launch(route_topk_kernel, (unsigned)((tokens + 3) / 4), 128, smem, stream, z, correction, chosen, weights, tokens, outputs, top,
-               sigmoid);
+               sigmoid, groups, keep, tiny);
     LLM_CHECK_LAUNCH("route_topk");
     return 0;
 }

@@ -103,13 +103,18 @@ _SIGNATURES = {
                                     _c_void_p],
     "llm_norm_add": [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p,
                      _c_void_p, _c_void_p],
+    "llm_add_dynamic_tanh": [_c_void_p, _c_void_p, _c_int, _c_int, ctypes.c_longlong, _c_void_p, _c_void_p, _c_int, _c_float, _c_void_p,
+                             _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, ctypes.c_longlong, _c_int, _c_int, _c_int, _c_void_p],
+    "llm_embed_dynamic_tanh": [_c_void_p, _c_void_p, _c_int, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int,
+                               ctypes.c_longlong, _c_int, _c_int, _c_int, _c_void_p],
+    "llm_softcap_f32": [_c_void_p, _c_float, ctypes.c_longlong, _c_void_p],
     "llm_rmsnorm_rows": [_c_void_p, ctypes.c_longlong, _c_void_p, ctypes.c_longlong, _c_void_p, _c_int, _c_int, _c_int, _c_float,
                          _c_void_p],
     "llm_glu_act": [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "llm_token_side_gate": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "llm_glu_clamped": [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_float, _c_void_p],
     "llm_latent_prepare": [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_float, _c_void_p, _c_void_p,
-                           _c_void_p, ctypes.c_longlong, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+                           _c_void_p, ctypes.c_longlong, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
     "llm_headnorm_store": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_void_p, ctypes.c_longlong, _c_int,
                            _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "llm_attention_flat": [_c_void_p, _c_int, _c_void_p, ctypes.c_longlong, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int,
@@ -142,7 +147,7 @@ _SIGNATURES = {
     "llm_gemm_grouped": [_c_void_p, ctypes.c_longlong, ctypes.c_longlong, ctypes.c_longlong, _c_void_p, _c_void_p, _c_void_p,
                          ctypes.c_longlong, ctypes.c_longlong, ctypes.c_longlong, _c_int, _c_int, _c_int, _c_int, _c_int,
                          _c_void_p, _c_int, _c_int, _c_float, _c_float, _c_void_p, _c_void_p, _c_void_p],
-    "llm_route_topk": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+    "llm_route_topk": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p],
     "llm_moe_plan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p,
                      _c_void_p, _c_void_p],
     "llm_gather_rows": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
@@ -198,6 +203,8 @@ class PartialSums:
     stream), `out` the tensor the sum belongs in.  `Kernels.add_rmsnorm` and `Kernels.rope_store` take it in
     place of the tensor and add the parts while they read; `sum()` adds them into `out` by a kernel of its own."""
 
+    taken_by = "takes_partial_sums"       # what a part's class sets to be handed one of these as it is
+
     def __init__(self, kernels, parts, out):
         self.k, self.parts, self.out = kernels, parts, out
         self.shape, self.dtype = out.shape, out.dtype
@@ -214,9 +221,25 @@ class PartialSums:
         return self.k.sum_parts(self.parts, self.out)
 
 
+class RoutedSum:
+    """The result of a routed feed-forward whose weighted sum over each token's choices is still to be taken: the experts'
+    output rows `y` sorted by expert, the sorted row of every (token, choice) pair, and the weights.  A kernel that adds a
+    branch to the stream takes it in place of the tensor (`Kernels.add_dynamic_tanh`); `sum()` adds it up by a kernel of
+    its own.  Valid until the next routed feed-forward of the step writes its rows."""
+
+    taken_by = "takes_routed_sums"
+
+    def __init__(self, kernels, y, plan, chosen, weights, x, experts, out):
+        self.k, self.y, self.plan, self.chosen, self.weights, self.x, self.experts, self.out = kernels, y, plan, chosen, weights, x, experts, out
+        self.shape, self.dtype = out.shape, out.dtype
+
+    def sum(self):
+        return self.k.moe_combine(self.y, self.plan, self.chosen, self.weights, self.x, self.experts, self.out)
+
+
 def materialize(x):
-    """The tensor of `x`, which may be a PartialSums."""
-    return x.sum() if isinstance(x, PartialSums) else x
+    """The tensor of `x`, which may be a PartialSums or a RoutedSum."""
+    return x if isinstance(x, torch.Tensor) else x.sum()
 
 
 class AttentionPlan:
@@ -474,6 +497,67 @@ class Kernels:
                    DTYPE_CODE[weight.dtype], _ptr(out), DTYPE_CODE[out.dtype], out.shape[0], width, float(eps),
                    splits, stride, self._stream())
         return out
+
+    def add_dynamic_tanh(self, residual, delta, factor: float, norm, out, rows=None, store: bool = True):
+        """residual += factor * delta (when given; kept only with `store` and without `rows`); out = tanh(alpha * residual[rows]) *
+        gain + shift with norm = (alpha [1], gain [width], shift [width]) float32, or with norm None the stream itself as out's
+        type.  `delta`: a tensor, a PartialSums or a RoutedSum; `out` may be a column range of a wider matrix; csrc/dynamic_tanh.cu."""
+        _check(residual, "add_dynamic_tanh.residual", torch.float32, 2)
+        width = residual.shape[1]
+        _need(out.dim() == 2 and out.is_cuda and out.dtype in DTYPE_CODE and out.stride(1) == 1 and out.shape[1] == width and
+              out.stride(0) >= width, "add_dynamic_tanh.out: rows of the stream's width in one of the engine's types")
+        alpha = gain = shift = None
+        if norm is not None:
+            alpha, gain, shift = norm
+            for name, v, n in (("alpha", alpha, 1), ("gain", gain, width), ("shift", shift, width)):
+                _check(v, "add_dynamic_tanh." + name, torch.float32, 1)
+                _need(v.shape[0] == n, f"add_dynamic_tanh.{name}: {n} numbers")
+        if rows is not None:
+            _check(rows, "add_dynamic_tanh.rows", torch.int32, 1)
+        _need(out.shape[0] == (residual if rows is None else rows).shape[0], "add_dynamic_tanh.out: one row per row asked for")
+        if isinstance(delta, PartialSums) and delta.splits > 8:
+            delta = delta.sum()
+        data, dtype, splits, stride, place, weights, top = None, 0, 0, 0, None, None, 0
+        if delta is not None:
+            _need(tuple(delta.shape) == tuple(residual.shape), "add_dynamic_tanh.delta: shape differs from residual")
+        if isinstance(delta, PartialSums):
+            data, splits, stride = delta.parts, delta.splits, delta.stride
+        elif isinstance(delta, RoutedSum):
+            data, dtype, place, weights, top = delta.y, DTYPE_CODE[delta.y.dtype], delta.plan["place"], delta.weights, delta.chosen.shape[1]
+        elif delta is not None:
+            _check(delta, "add_dynamic_tanh.delta", tuple(DTYPE_CODE), 2)
+            data, dtype = delta, DTYPE_CODE[delta.dtype]
+        self._call("llm_add_dynamic_tanh", _ptr(residual), _ptr(data), dtype, splits, stride, _ptr(place), _ptr(weights), top, float(factor),
+                   _ptr(rows), _ptr(alpha), _ptr(gain), _ptr(shift), out.data_ptr(), DTYPE_CODE[out.dtype], out.stride(0), out.shape[0],
+                   width, 1 if store and rows is None and delta is not None else 0, self._stream())
+        return out
+
+    def embed_dynamic_tanh(self, ids, table, scale: float, norm, out, cast_out=None):
+        """out[t] = tanh(alpha * scale * table[ids[t]]) * gain + shift as float32, norm = (alpha, gain, shift); `cast_out`: the same rows
+        in another type (may be a column range of a wider matrix)."""
+        _check(ids, "embed_dynamic_tanh.ids", torch.int32, 1)
+        _check(table, "embed_dynamic_tanh.table", tuple(DTYPE_CODE), 2)
+        _check(out, "embed_dynamic_tanh.out", torch.float32, 2)
+        width = table.shape[1]
+        _need(out.shape == (ids.shape[0], width), "embed_dynamic_tanh.out: wrong shape")
+        alpha, gain, shift = norm
+        for name, v, n in (("alpha", alpha, 1), ("gain", gain, width), ("shift", shift, width)):
+            _check(v, "embed_dynamic_tanh." + name, torch.float32, 1)
+            _need(v.shape[0] == n, f"embed_dynamic_tanh.{name}: {n} numbers")
+        if cast_out is not None:
+            _need(cast_out.is_cuda and cast_out.dtype in DTYPE_CODE and tuple(cast_out.shape) == tuple(out.shape) and
+                  cast_out.stride(1) == 1 and cast_out.stride(0) >= width, "embed_dynamic_tanh.cast_out: rows like out")
+        self._call("llm_embed_dynamic_tanh", _ptr(ids), _ptr(table), DTYPE_CODE[table.dtype], float(scale), _ptr(alpha), _ptr(gain), _ptr(shift),
+                   _ptr(out), cast_out.data_ptr() if cast_out is not None else None,
+                   DTYPE_CODE[cast_out.dtype] if cast_out is not None else 0, cast_out.stride(0) if cast_out is not None else 0,
+                   ids.shape[0], width, table.shape[0], self._stream())
+        return out
+
+    def softcap_(self, x, cap: float):
+        """x = cap * tanh(x / cap), float32, in place."""
+        _check(x, "softcap_.x", torch.float32)
+        self._call("llm_softcap_f32", _ptr(x), float(cap), x.numel(), self._stream())
+        return x
 
     def rope_tables(self, positions, inv_freq, cos, sin, amplitude: float = 1.0):
         """cos[t, i] = amplitude * cos(positions[t] * inv_freq[i]) and sin likewise, float32 [tokens, rotary_dim/2]."""
@@ -909,11 +993,14 @@ class Kernels:
                    _ptr(out_gate), self._stream())
         return out
 
-    def route_topk(self, scores, correction, chosen, weights, sigmoid: bool = False, chosen_softmax: bool = False):
+    def route_topk(self, scores, correction, chosen, weights, sigmoid: bool = False, chosen_softmax: bool = False, groups=None,
+                   renormalize: float | None = None):
         """Router outputs [T, R] float32 -> chosen [T, top] int32 (the largest s + correction, descending; correction None: of
         s) and weights [T, top] float32 (their s), where s is the softmax over the outputs, or with `sigmoid` each output's
         sigmoid.  `chosen_softmax`: the outputs themselves are compared, plus `correction` as a bias that belongs to them, and
-        the weights are the softmax over the chosen outputs alone; csrc/moe_route.cu."""
+        the weights are the softmax over the chosen outputs alone.  `groups` = (count, keep): the outputs form `count` equal groups
+        of neighbours and only those of the `keep` groups with the largest single entry can be chosen.  `renormalize` = tiny: the
+        weights are divided by their sum plus that; csrc/moe_route.cu."""
         _check(scores, "route_topk.scores", torch.float32, 2)
         if correction is not None:
             _check(correction, "route_topk.correction", torch.float32, 1)
@@ -922,8 +1009,10 @@ class Kernels:
         tokens, outputs = scores.shape
         _need((correction is None or correction.shape[0] == outputs) and chosen.shape[0] == tokens and
               tuple(weights.shape) == tuple(chosen.shape), "route_topk: shapes do not fit")
+        count, keep = groups if groups else (1, 1)
+        _need(renormalize is None or renormalize > 0, "route_topk: renormalize adds a positive number to the sum")
         self._call("llm_route_topk", _ptr(scores), _ptr(correction), _ptr(chosen), _ptr(weights), tokens, outputs, chosen.shape[1],
-                   2 if chosen_softmax else 1 if sigmoid else 0, self._stream())
+                   2 if chosen_softmax else 1 if sigmoid else 0, int(count), int(keep), float(renormalize or 0.0), self._stream())
 
     def moe_tile_bound(self, rows: int, experts: int) -> int:
         """The most row tiles `moe_plan` can make of `rows` (token, choice) pairs over `experts` experts."""
@@ -972,24 +1061,28 @@ class Kernels:
     def moe_linear(self, a, w, out, plan, gather: bool = False, glu=False, limit: float = 0.0, slope: float = 1.0):
         """out[r] = a[row of r] . w[expert of r]^T for every sorted row r of `plan`; with `gather` a's rows are tokens
         (read through plan["source"]), else sorted rows.  `glu`: w [E, 2n, k] holds gate rows then up rows and the gate is
-        applied in the epilogue: True or "clamped" the clamped form (limit, slope), "silu_weighted" silu(w g) * (w u) with
-        the plan's weight w of the row (the expert's product of the row times w)."""
+        applied in the epilogue: True or "clamped" the clamped form (limit, slope), "silu" silu(g) * u, "silu_weighted"
+        silu(w g) * (w u) with the plan's weight w of the row (the expert's product of the row times w)."""
         _check(a, "moe_linear.a", tuple(DTYPE_CODE), 2)
         _check(w, "moe_linear.w", a.dtype, 3)
         _check(out, "moe_linear.out", a.dtype, 2)
         experts, wn, k = w.shape
         n = wn // 2 if glu else wn
         _need(a.shape[1] == k and out.shape[1] == n and out.shape[0] == plan["source"].shape[0], "moe_linear: shapes do not fit")
-        form = 0 if not glu else 2 if glu == "silu_weighted" else 1
-        _need(form != 2 or plan.get("row_weight") is not None, "moe_linear: the plan holds no row weights")
+        form = 0 if not glu else 2 if glu in ("silu", "silu_weighted") else 1
+        weighted = glu == "silu_weighted"
+        _need(not weighted or plan.get("row_weight") is not None, "moe_linear: the plan holds no row weights")
         self._call("llm_gemm_grouped", _ptr(a), a.shape[1], 0, 0, _ptr(plan["source"]) if gather else None, _ptr(w), _ptr(out),
                    out.shape[1], 0, 0, DTYPE_CODE[a.dtype], 0, n, k, experts, _ptr(plan["tiles"]), plan["bound"],
-                   form, float(limit), float(slope), _ptr(plan["row_weight"]) if form == 2 else None, None, self._stream())
+                   form, float(limit), float(slope), _ptr(plan["row_weight"]) if weighted else None, None, self._stream())
         return out
 
-    def moe_combine(self, y, plan, chosen, weights, x, experts: int, out):
+    def moe_combine(self, y, plan, chosen, weights, x, experts: int, out, defer: bool = False):
         """out[t] = sum_j weights[t, j] * (y[sorted row of (t, j)], or x[t] where chosen[t, j] >= experts), j in order;
-        weights None: all 1."""
+        weights None: all 1.  With `defer` nothing is launched and a RoutedSum comes back (the caller's next kernel adds
+        the rows as it reads; only where every choice has an expert's row)."""
+        if defer:
+            return RoutedSum(self, y, plan, chosen, weights, x, experts, out)
         _check(x, "moe_combine.x", tuple(DTYPE_CODE), 2)
         _check(out, "moe_combine.out", x.dtype, 2)
         _check(chosen, "moe_combine.chosen", torch.int32, 2)
@@ -1015,25 +1108,31 @@ class Kernels:
         return cache_layer.shape[1] // per_token
 
     def latent_prepare(self, qd, tables, rotary_dim, interleaved, gain, eps, q_out, cache_layer, slots, heads, dim, rot_dim, rank,
-                       kv=None):
+                       kv=None, gate_out=None):
         """From the fused projection qd [T, heads * (dim + rot_dim) + rank + rot_dim]: the latent part normed (gain [rank]
         float32) and the shared key part rotated, stored together as one cache row per token at `slots` (None: no store);
         every head's rotated query part written to q_out [T, heads * (rank + rot_dim)] behind the place of its absorbed
         part.  tables = (cos, sin) float32 [T, rotary_dim / 2]; csrc/attention_flat.cu.  With `kv` [T, rank + rot_dim] (rows
-        with a stride of their own: columns of another product) qd holds the queries alone."""
+        with a stride of their own: columns of another product) qd holds the queries alone.  With `gate_out` [T, heads] float32 the
+        row goes on with a gate's number per head (and any padding behind them), which are copied there."""
         _check(qd, "latent_prepare.qd", tuple(DTYPE_CODE), 2)
         _check(q_out, "latent_prepare.q_out", qd.dtype, 2)
         _check(gain, "latent_prepare.gain", torch.float32, 1)
         tokens = qd.shape[0]
         qw = heads * (dim + rot_dim)
         if kv is None:
-            _need(qd.shape[1] == qw + rank + rot_dim, "latent_prepare.qd: wrong width")
+            extra = qd.shape[1] - (qw + rank + rot_dim)
+            _need(extra == 0 if gate_out is None else extra >= heads, "latent_prepare.qd: wrong width")
             kv_ptr, ld_kv = qd.data_ptr() + qw * qd.element_size(), qd.shape[1]
         else:
+            _need(gate_out is None, "latent_prepare: a gate's numbers lie behind the shared key part of the fused projection")
             _need(kv.dim() == 2 and kv.dtype == qd.dtype and kv.is_cuda and kv.stride(1) == 1 and
                   tuple(kv.shape) == (tokens, rank + rot_dim) and qd.shape[1] == qw, "latent_prepare.kv: [tokens, rank + rot_dim] beside queries alone")
             kv_ptr, ld_kv = kv.data_ptr(), kv.stride(0)
         _need(gain.shape[0] == rank and tuple(q_out.shape) == (tokens, heads * (rank + rot_dim)), "latent_prepare: shapes do not fit")
+        if gate_out is not None:
+            _check(gate_out, "latent_prepare.gate_out", torch.float32, 2)
+            _need(tuple(gate_out.shape) == (tokens, heads), "latent_prepare.gate_out: [tokens, heads]")
         cos = sin = None
         if rotary_dim:
             cos, sin = tables
@@ -1048,7 +1147,7 @@ class Kernels:
             page_size, stride = self._flat_page_size(cache_layer, 1, rank + rot_dim, rank, True), cache_layer.shape[1]
         self._call("llm_latent_prepare", _ptr(qd), qd.shape[1], kv_ptr, ld_kv, _ptr(cos), _ptr(sin), int(rotary_dim), 1 if interleaved else 0,
                    _ptr(gain), float(eps), _ptr(q_out), _ptr(cache_layer) if slots is not None else None, _ptr(slots), stride,
-                   page_size, DTYPE_CODE[qd.dtype], tokens, heads, dim, rot_dim, rank, self._stream())
+                   page_size, DTYPE_CODE[qd.dtype], tokens, heads, dim, rot_dim, rank, _ptr(gate_out), self._stream())
 
     def headnorm_store(self, qkv, q_gain, k_gain, eps, cache_layer, slots, heads, kv_heads, dim, vdim):
         """qkv [T, heads * dim + kv_heads * (dim + vdim)]: every query head (in place) and key head divided by its root

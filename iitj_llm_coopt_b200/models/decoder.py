@@ -13,6 +13,7 @@ import torch
 
 from .. import parts as P
 from ..parts.base import delta_for
+from ..parts.stream_join import ORIGIN
 
 
 def _lookup(family: str, spec, what: str):
@@ -49,6 +50,9 @@ def model_parameter_specs(spec) -> dict:
                 out[f"layers.{i}.{part_name}.{pname}"] = pspec
     for pname, pspec in _lookup("norm", spec.final_norm, "norm").parameters(spec.final_norm).items():
         out[f"final_norm.{pname}"] = pspec
+    if spec.join is not None:
+        for pname, pspec in _lookup("stream_join", spec.join, "stream join").parameters(spec.join).items():
+            out[f"stream_join.{pname}"] = pspec
     head = spec.head_spec()
     head_cls = _lookup("head", head, "head")
     for pname, pspec in head_cls.parameters(head).items():
@@ -112,14 +116,20 @@ class DecoderModel:
             self.layers.append(block)
         self.final_norm = build_part("norm", spec.final_norm, _lookup("norm", spec.final_norm, "norm"), kernels, dtype, device,
                                      "final_norm")
+        self.join = None
+        if spec.join is not None:
+            self.join = build_part("stream_join", spec.join, _lookup("stream_join", spec.join, "stream join"), kernels, dtype, device,
+                                   "stream_join")
+        elif any(call.join for call in spec.order):
+            raise ValueError("the run order joins the embedding's output to the stream, but the model names no stream join")
         head = spec.head_spec()
         self.head = build_part("head", head, _lookup("head", head, "head"), kernels, dtype, device)
 
     def all_parts(self) -> list:
         """Every part of the model, the parts that parts own included (each object once)."""
         seen, out = set(), []
-        for part in [self.embedding] + [p for b in self.layers for p in b.all_parts()] + [self.final_norm, self.head]:
-            if id(part) not in seen:
+        for part in [self.embedding] + [p for b in self.layers for p in b.all_parts()] + [self.join, self.final_norm, self.head]:
+            if part is not None and id(part) not in seen:
                 seen.add(id(part))
                 out.append(part)
         return out
@@ -142,6 +152,8 @@ class DecoderModel:
             per_part.setdefault(owner, {})[name] = t
         self.embedding.load(per_part["embedding"])
         self.final_norm.load(per_part["final_norm"])
+        if self.join is not None:
+            self.join.load(per_part["stream_join"])
         head_params = dict(per_part.get("lm_head", {}))
         tied = getattr(self.head, "tied_parameter", None)
         if self.spec.tie_embeddings and tied is not None:
@@ -164,8 +176,14 @@ class DecoderModel:
     def forward(self, ctx):
         """Runs the tokens of `ctx` through the model; returns float32 logits [ctx.num_logits, vocab]
         for the rows in ctx.logit_rows (None if no row is wanted)."""
+        if self.join is not None:
+            ctx.shared[ORIGIN] = self.join.origin(ctx)          # an embedding that knows how leaves its rows there
         residual, delta = self.embedding.forward(ctx), None
+        if self.join is not None and ctx.shared.pop(ORIGIN, None) is not None:
+            self.join.keep(ctx, residual)
         for call in self.spec.order:
+            if call.join:
+                residual, delta = self.join.forward(ctx, residual, delta_for(self.join, delta)), None
             residual, delta = self.layers[call.layer].forward(ctx, residual, delta, call)
         if ctx.num_logits == 0:
             return None

@@ -10,7 +10,7 @@ from __future__ import annotations
 from .base import ParamSpec, Part, StepPlan, StepShape
 from .block import (Arrangement, BranchNormBlock, BranchNormMixerBlock, PostNormDepthBlock, PostNormDepthMixerBlock, PreNormBlock,
                     PreNormMixerBlock, SandwichBlock, SandwichMixerBlock, SandwichMixerSideBlock, SandwichSideBlock)
-from .embedding import Embedding, NormedEmbedding, OutputHead, SideTableEmbedding
+from .embedding import Embedding, NormedEmbedding, OutputHead, SideTableEmbedding, TanhNormedEmbedding
 from .feed_forward import GLU, ClampedGLU, PolyNormMLP, RoutedGLU, SwiGLU
 from .gated_attention import GatedAttention
 from .latent_attention import LatentAttention
@@ -18,14 +18,16 @@ from .lru import GatedLRU
 from .mixer import PagedAttention
 from .parallel import ParallelMixer
 from .retention import Retention
+from .stream_join import StreamJoin
 from .stream_mix import DepthAverage
 from .talking_attention import TalkingAttention
 from .token_input import GatedTableInput
 from .wkv import WKV
-from .norm import OnePlusRMSNorm, RMSNorm, ScalarGainRMSNorm
+from .norm import DynamicTanh, OnePlusRMSNorm, RMSNorm, ScalarGainRMSNorm
 from .position import NoPosition, RotaryEmbedding, rope_inverse_frequencies
 
-NORMS = {"rmsnorm": RMSNorm, "rmsnorm_scalar": ScalarGainRMSNorm, "rmsnorm_one_plus": OnePlusRMSNorm}
+NORMS = {"rmsnorm": RMSNorm, "rmsnorm_scalar": ScalarGainRMSNorm, "rmsnorm_one_plus": OnePlusRMSNorm,
+         "dynamic_tanh": DynamicTanh}
 POSITION_ENCODINGS = {"rope": RotaryEmbedding, "none": NoPosition}
 MIXERS = {"attention": PagedAttention, "talking_attention": TalkingAttention, "retention": Retention,
           "latent_attention": LatentAttention, "gated_attention": GatedAttention, "wkv": WKV, "gated_lru": GatedLRU,
@@ -35,14 +37,17 @@ ARRANGEMENTS = {"prenorm": PreNormBlock, "prenorm_mixer": PreNormMixerBlock, "br
                 "branchnorm_mixer": BranchNormMixerBlock, "sandwich": SandwichBlock, "sandwich_mixer": SandwichMixerBlock,
                 "sandwich_side": SandwichSideBlock, "sandwich_mixer_side": SandwichMixerSideBlock,
                 "postnorm_depth": PostNormDepthBlock, "postnorm_depth_mixer": PostNormDepthMixerBlock}
-EMBEDDINGS = {"table": Embedding, "table_norm": NormedEmbedding, "table_side": SideTableEmbedding}
+EMBEDDINGS = {"table": Embedding, "table_norm": NormedEmbedding, "table_side": SideTableEmbedding,
+              "table_dynamic_tanh": TanhNormedEmbedding}
 TOKEN_INPUTS = {"gated_table": GatedTableInput}
 STREAM_MIXES = {"depth_average": DepthAverage}
+STREAM_JOINS = {"concat": StreamJoin}
 HEADS = {"linear": OutputHead}
 
 # family name (what an arrangement's PARTS declares for a part name) -> registry
 FAMILIES = {"norm": NORMS, "mixer": MIXERS, "feed_forward": FEED_FORWARDS, "position": POSITION_ENCODINGS,
-            "embedding": EMBEDDINGS, "head": HEADS, "token_input": TOKEN_INPUTS, "stream_mix": STREAM_MIXES}
+            "embedding": EMBEDDINGS, "head": HEADS, "token_input": TOKEN_INPUTS, "stream_mix": STREAM_MIXES,
+            "stream_join": STREAM_JOINS}
 
 
 def register_norm(kind, cls):
@@ -79,3 +84,7 @@ def register_token_input(kind, cls):
 
 def register_stream_mix(kind, cls):
     STREAM_MIXES[kind] = cls
+
+
+def register_stream_join(kind, cls):
+    STREAM_JOINS[kind] = cls

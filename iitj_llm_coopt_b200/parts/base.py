@@ -17,6 +17,8 @@ Interfaces (T = tokens of the step, w = model width):
   Mixer.forward(ctx, x[T,w], call) -> delta[T,w];  Mixer.cache_need() -> CacheNeed
   FeedForward.forward(ctx, x[T,w]) -> delta[T,w]
   Embedding.forward(ctx) -> residual[T,w] f32;   Head.forward(ctx, x[N,w]) -> logits[N,vocab] f32
+  StreamJoin.forward(ctx, residual, delta) -> residual (before a call whose `join` is set);  origin(ctx), keep(ctx, residual):
+      where the embedding's rows are kept for it (parts/stream_join.py)
   Arrangement.forward(ctx, residual, delta, call) -> (residual, delta)     (parts/block.py)
 
 Per-step index arrays of a part's own.  The step function builds the arrays every part needs (positions, block
@@ -34,6 +36,8 @@ that was split along k and whose parts are still to be added.  It is only handed
 encoding whose class sets `takes_partial_sums = True` (the built-in ones pass it on to kernels that add the
 parts while they read); for any other part `delta_for(part, delta)` adds them first.  The parts live in
 scratch that the next split product overwrites, so an arrangement uses a delta before it runs another product.
+A routed feed-forward hands on a `kernels.RoutedSum` (its weighted sum over each token's choices still to be taken) in the
+same way; a part that adds it up itself sets `takes_routed_sums = True`.
 """
 from __future__ import annotations
 
@@ -43,8 +47,8 @@ import torch
 
 
 def delta_for(part, delta):
-    """`delta` as `part` can take it: partial sums are added now unless the part adds them itself."""
-    if delta is not None and not isinstance(delta, torch.Tensor) and not getattr(part, "takes_partial_sums", False):
+    """`delta` as `part` can take it: sums still to be taken are taken now unless the part takes them itself."""
+    if delta is not None and not isinstance(delta, torch.Tensor) and not getattr(part, delta.taken_by, False):
         return delta.sum()
     return delta
 

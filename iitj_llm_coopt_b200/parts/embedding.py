@@ -2,7 +2,7 @@
 
 `Embedding`: x = table[token_ids] (engine/model.py:191), written as the float32 residual stream.
 `OutputHead`: logits = x . W^T in float32 (engine/model.py:215-218); W is the embedding table
-when the model ties them (engine/model.py:106).
+when the model ties them (engine/model.py:106).  The spec's option `softcap` c > 0 caps them: c tanh(logits / c).
 """
 from __future__ import annotations
 
@@ -54,6 +54,32 @@ class NormedEmbedding(Embedding):
         return out
 
 
+class TanhNormedEmbedding(Embedding):
+    """x = tanh(alpha * scale * table[token_ids]) * norm + bias, the norm without statistics (parts/norm.py: DynamicTanh) on the
+    looked-up rows, in one kernel.  Where the model joins the embedding's rows to the stream later on (parts/stream_join.py), the
+    kernel leaves them there as the engine's type on the way."""
+
+    def __init__(self, spec, kernels, dtype=None):
+        super().__init__(spec, kernels, dtype)
+        self.norm = self.bias = self.alpha = None
+
+    @classmethod
+    def parameters(cls, spec) -> dict:
+        return {"weight": ParamSpec((spec.vocab, spec.width), kind="table"), "norm": ParamSpec((spec.width,), kind="vector"),
+                "bias": ParamSpec((spec.width,), kind="vector"), "alpha": ParamSpec((), kind="vector")}
+
+    def load(self, tensors: dict) -> None:
+        self.weight = tensors["weight"]
+        self.norm, self.bias = tensors["norm"].float().contiguous(), tensors["bias"].float().contiguous()
+        self.alpha = tensors["alpha"].float().reshape(1).contiguous()
+
+    def forward(self, ctx):
+        from .stream_join import ORIGIN
+        out = ctx.buffer("residual", (ctx.num_tokens, self.width), torch.float32)
+        return self.k.embed_dynamic_tanh(ctx.token_ids, self.weight, self.scale, (self.alpha, self.norm, self.bias), out,
+                                         cast_out=ctx.shared.pop(ORIGIN, None))
+
+
 class SideTableEmbedding(Embedding):
     """x = table[token_ids], and a second table [vocab, side_width] (option `side_width`) whose rows the layers' token
     inputs read by the same ids: it is left in `ctx.shared` for them every step (parts/token_input.py)."""
@@ -80,6 +106,7 @@ class OutputHead(Part):
 
     def __init__(self, spec, kernels, dtype=None):
         self.spec, self.vocab, self.width, self.k, self.scale = spec, spec.vocab, spec.width, kernels, spec.scale
+        self.softcap = float(dict(spec.options).get("softcap", 0.0))
         self.weight = None
 
     @classmethod
@@ -91,4 +118,6 @@ class OutputHead(Part):
         self.k.linear(x, self.weight, logits)
         if self.scale != 1.0:
             self.k.scale_(logits, self.scale)
+        if self.softcap > 0.0:
+            self.k.softcap_(logits, self.softcap)
         return logits

@@ -135,14 +135,17 @@ class RoutedGLU(Part):
     `router` = "chosen_softmax" compares the router outputs themselves and takes the softmax over the chosen ones alone as weights
     (they sum to one); `router_bias` = True adds a stored bias to the router outputs before anything else;
     `correction` = False: there is no stored correction and the choice is by s alone; `expert` = "silu" makes the
-    experts plain silu-gated ones, silu(g) * u, instead of the clamped form; `weight_on` = "input" feeds expert e the row
+    experts plain silu-gated ones, silu(g) * u, instead of the clamped form; `groups` = (count, keep): the router outputs form
+    `count` equal groups of neighbours and only those of the `keep` groups with the largest single score can be chosen;
+    `renormalize` = tiny: the chosen scores are divided by (their sum + tiny); `weight_on` = "input" feeds expert e the row
     s[e] * x and sums the experts' outputs as they are, out = sum expert_e(s[e] * x) (the first product being linear in
     its row, the weight is applied to gate and up in that product's epilogue, or to the gathered rows).
 
     The last `identity` router outputs stand for experts without tensors that hand their input back (s[e] * x).
     Rows are sorted by expert on the device (`Kernels.moe_plan`), the experts' products run as one grouped product each
     (the first reads its rows through the sorted index, applies the gate in its epilogue), and the chosen experts'
-    outputs of a token are added in the order of its choices, so a token's result does not depend on the batch.
+    outputs of a token are added in the order of its choices, so a token's result does not depend on the batch; without
+    identity experts that sum is left to whatever adds the result to the stream (`kernels.RoutedSum`).
     Nothing of that comes back to the host, so decode steps replay from CUDA graphs.  A step with many rows (a prompt
     portion; `Kernels.moe_dense_rows`) that is not being captured reads the experts' row counts once and runs each
     expert's rows, gathered side by side, through the dense product kernels, which are several times faster at that size."""
@@ -168,8 +171,15 @@ class RoutedGLU(Part):
             raise ValueError("routed feed-forward: router is softmax or sigmoid, weight_on is input or output")
         if self.on_input and (self.identity or not self.silu):
             raise ValueError("routed feed-forward: weights on the experts' inputs go with plain silu experts and no identity experts")
-        if self.silu and not self.on_input:
-            raise ValueError("routed feed-forward: plain silu experts are served with the weight on their input")
+        groups = spec.option("groups")
+        self.groups = (int(groups[0]), int(groups[1])) if groups else None
+        self.renormalize = spec.option("renormalize")
+        outputs = self.experts + self.identity
+        if self.groups and (outputs % self.groups[0] or not 1 <= self.groups[1] <= self.groups[0] or
+                            self.top > outputs // self.groups[0] * self.groups[1]):
+            raise ValueError(f"routed feed-forward: {self.top} of {outputs} router outputs from groups {self.groups}")
+        if self.chosen_softmax and (self.renormalize is not None or self.groups):
+            raise ValueError("routed feed-forward: router = chosen_softmax takes neither groups nor a renormalisation")
         self.router = self.correction = self.router_bias = self.expert_gate_up = self.expert_down = None
         self.prepare_key = f"routed_glu.{self.top}"          # layers with as many choices a token share the step's plan
 
@@ -217,7 +227,8 @@ class RoutedGLU(Part):
         if self.chosen_softmax:
             self.k.route_topk(scores, self.router_bias, chosen, weights, chosen_softmax=True)
         else:
-            self.k.route_topk(scores, self.correction, chosen, weights, sigmoid=self.sigmoid)
+            more = {} if not self.groups and self.renormalize is None else {"groups": self.groups, "renormalize": self.renormalize}
+            self.k.route_topk(scores, self.correction, chosen, weights, sigmoid=self.sigmoid, **more)
         out = ctx.buffer("ffn.out", (t, self.width), self.dtype)
         plan = y = None
         if self.experts:
@@ -253,7 +264,9 @@ class RoutedGLU(Part):
                     if hi > lo:
                         self.k.linear(act[lo:hi], w2[e], y[lo:hi])
             else:
-                self.k.moe_linear(x, w1, act, plan, gather=True, glu="silu_weighted" if self.silu else True, limit=self.limit,
+                glu = ("silu_weighted" if self.on_input else "silu") if self.silu else True
+                self.k.moe_linear(x, w1, act, plan, gather=True, glu=glu, limit=self.limit,
                                   slope=self.slope)
                 self.k.moe_linear(act, w2, y, plan)
-        return self.k.moe_combine(y, plan, chosen, None if self.on_input else weights, x, self.experts, out)
+        return self.k.moe_combine(y, plan, chosen, None if self.on_input else weights, x, self.experts, out,
+                                  **({"defer": True} if self.experts and not self.identity else {}))

@@ -313,14 +313,34 @@ def ref_attention_flat(q, q_stride_heads, cache, block_table, token_request, pos
     return out.view(T, heads * value_dim)
 
 
-def ref_route_topk(scores, correction, top, sigmoid=False, chosen_softmax=False):
+def ref_route_topk(scores, correction, top, sigmoid=False, chosen_softmax=False, groups=None, renormalize=None):
     if chosen_softmax:             # the outputs (plus their bias) compared as they are; softmax over the chosen alone
         z = scores.float() + (correction.float() if correction is not None else 0.0)
         val, chosen = torch.topk(z, top, dim=-1)
         return chosen.to(torch.int32), torch.softmax(val, dim=-1)
     s = torch.sigmoid(scores.float()) if sigmoid else torch.softmax(scores.float(), dim=-1)
-    chosen = torch.topk(s + correction.float() if correction is not None else s, top, dim=-1).indices
-    return chosen.to(torch.int32), torch.gather(s, 1, chosen)
+    c = s + correction.float() if correction is not None else s
+    if groups:                     # only entries of the groups with the largest single entry can be chosen
+        count, keep = groups
+        parts = c.view(c.shape[0], count, -1)
+        best = torch.topk(parts.amax(-1), keep, dim=-1).indices
+        shut = torch.ones(c.shape[0], count, dtype=torch.bool, device=c.device).scatter_(1, best, False)
+        c = parts.masked_fill(shut.unsqueeze(-1), float("-inf")).reshape(c.shape)
+    chosen = torch.topk(c, top, dim=-1).indices
+    w = torch.gather(s, 1, chosen)
+    if renormalize is not None:
+        w = w / (w.sum(-1, keepdim=True) + renormalize)
+    return chosen.to(torch.int32), w
+
+
+# ---- the Bidinex family's kernels ------------------------------------------------------------------------------
+
+def ref_dynamic_tanh(x, norm):
+    """tanh(alpha x) * gain + shift, norm = (alpha [1], gain, shift); None: x itself."""
+    if norm is None:
+        return x.float()
+    alpha, gain, shift = norm
+    return torch.tanh(alpha.float() * x.float()) * gain.float() + shift.float()
 
 
 def ref_qk_prepare(proj, heads, kv_heads, dim, vdim, eps, bias=None, norm="none", q_gain=None, k_gain=None, norm_first=True,
@@ -510,6 +530,22 @@ class TorchKernels:
         out.copy_(y)
         return out
 
+    def add_dynamic_tanh(self, residual, delta, factor, norm, out, rows=None, store=True):
+        v = residual + factor * delta.float() if delta is not None else residual
+        if store and rows is None and delta is not None:
+            residual.copy_(v)
+        out.copy_(ref_dynamic_tanh(v if rows is None else v[rows.long()], norm))
+        return out
+
+    def embed_dynamic_tanh(self, ids, table, scale, norm, out, cast_out=None):
+        out.copy_(ref_dynamic_tanh(ref_embed(ids, table, scale), norm))
+        if cast_out is not None:
+            cast_out.copy_(out)
+        return out
+
+    def softcap_(self, x, cap):
+        return x.copy_(cap * torch.tanh(x / cap))
+
     def rope_tables(self, positions, inv_freq, cos, sin, amplitude=1.0):
         ang = positions.float().unsqueeze(1) * inv_freq.float().unsqueeze(0)
         cos.copy_(ang.cos() * amplitude)
@@ -616,7 +652,12 @@ class TorchKernels:
             out[:, out_offset + g * out_stride:out_offset + g * out_stride + n] = y
         return out
 
-    def latent_prepare(self, qd, tables, rotary_dim, interleaved, gain, eps, q_out, cache, slots, heads, dim, rot_dim, rank, kv=None):
+    def latent_prepare(self, qd, tables, rotary_dim, interleaved, gain, eps, q_out, cache, slots, heads, dim, rot_dim, rank, kv=None,
+                       gate_out=None):
+        if gate_out is not None:       # the gate's numbers lie behind the shared key part
+            at = heads * (dim + rot_dim) + rank + rot_dim
+            gate_out.copy_(qd[:, at:at + heads])
+            qd = qd[:, :at]
         cos, sin = tables if tables is not None else (None, None)
         qr, rows = ref_latent_prepare(qd, cos, sin, rotary_dim, interleaved, gain, eps, heads, dim, rot_dim, rank, kv)
         T = qd.shape[0]
@@ -685,8 +726,8 @@ class TorchKernels:
                           state, state_slots, cu_seqlens, write))
         return out
 
-    def route_topk(self, scores, correction, chosen, weights, sigmoid=False, chosen_softmax=False):
-        c, w = ref_route_topk(scores, correction, chosen.shape[1], sigmoid, chosen_softmax)
+    def route_topk(self, scores, correction, chosen, weights, sigmoid=False, chosen_softmax=False, groups=None, renormalize=None):
+        c, w = ref_route_topk(scores, correction, chosen.shape[1], sigmoid, chosen_softmax, groups, renormalize)
         chosen.copy_(c)
         weights.copy_(w)
 
@@ -737,12 +778,14 @@ class TorchKernels:
             y = a[rows].float() @ w[e].float().t()
             if glu == "silu_weighted":
                 y = ref_glu_act(y * plan["row_weight"][r0:r0 + n].unsqueeze(1), "silu")
+            elif glu == "silu":
+                y = ref_glu_act(y, "silu")
             elif glu:
                 y = ref_glu_clamped(y, limit, slope)
             out[r0:r0 + n] = y
         return out
 
-    def moe_combine(self, y, plan, chosen, weights, x, experts, out):
+    def moe_combine(self, y, plan, chosen, weights, x, experts, out, defer=False):     # always summed at once
         T, top = chosen.shape
         acc = torch.zeros(T, x.shape[1], dtype=torch.float32, device=x.device)
         for t in range(T):
