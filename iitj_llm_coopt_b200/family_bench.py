@@ -679,6 +679,136 @@ def _kernels_alone_mamusun(cfg, rod, tokens, batch, context, hbm_gbs, flush):
     return out
 
 
+def _kernels_alone_bidinex(cfg, beside, tokens, batch, context, hbm_gbs, flush):
+    """The kernels and kernel options that Bidinex brought, alone at the shapes of a `tokens`-token prompt and of a decode step of
+    `batch` requests, each beside the like kernel as Fomerax, Rodapel or Llama runs it at the same shape: microseconds, the bytes that
+    must move and the fraction of the copy bandwidth that is, or for arithmetic-bound kernels the TFLOP/s."""
+    import torch
+
+    from . import kernels as _k
+    from .parts.base import StepShape
+    from .parts.flat_tiles import plan_flat_tiles
+    K = _k.load()
+    dev, bf = "cuda", torch.bfloat16
+    m, mlp, width, vocab = cfg["layers"][0]["mixer"], cfg["layers"][0]["mlp"], cfg["width"], cfg["vocab"]
+    H, D, R, V, C = (m[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank"))
+    E, top, ff = mlp["router"]["experts"], mlp["router"]["top"], mlp["expert"]["ff"]
+    groups = (mlp["router"]["groups"]["count"], mlp["router"]["groups"]["keep"])
+    row, page, out = C + R, 16, []
+
+    def i32(x):
+        return torch.tensor(x, dtype=torch.int32, device=dev)
+
+    def rand(*shape, s=1.0):
+        return (torch.randn(*shape, device=dev) * s).to(bf)
+
+    def record(name, fn, nbytes=None, flops=None, like=None, reps=10):
+        us = 1e3 * _timed(fn, reps, 3, flush)
+        r = {"kernel": name, "us": round(us, 2)}
+        if nbytes is not None:
+            r.update(mbytes=round(nbytes / 1e6, 2), frac_of_copy_bandwidth=round(nbytes / (us * 1e-6) / (hbm_gbs * 1e9), 3))
+        if flops is not None:
+            r.update(tflops=round(flops / (us * 1e-6) / 1e12, 1))
+        if like:
+            r["like"] = like
+        out.append(r)
+
+    for label, T, B, per in (("prefill", tokens, 1, tokens), ("decode", batch, batch, 1)):
+        ctx_len = per if label == "prefill" else context
+        pages_per = -(-ctx_len // page)
+        treq = [b for b in range(B) for _ in range(per)]
+        pos = [ctx_len - per + i for _ in range(B) for i in range(per)]
+        table = torch.arange(B * pages_per, dtype=torch.int32, device=dev).view(B, pages_per)
+        slots = i32([int(table[b, p // page]) * page + p % page for b, p in zip(treq, pos)])
+        meta = SimpleNamespace(block_table=table, token_request=i32(treq), positions=i32(pos), query_lens=[per] * B,
+                               seq_lens_host=[ctx_len] * B, attention_plan=None)
+        causal = sum(p + 1 for p in pos)
+        # --- latent attention: the gate's numbers beside the latent row, the gate on the heads' sums of latent rows
+        pad = -(-H // 8) * 8
+        q_cols = H * (D + R)
+        qd_g, qd = rand(T, q_cols + row + pad), rand(T, q_cols + row)
+        cache, lgain = rand(B * pages_per + 1, page * row, s=0.5), torch.ones(C, device=dev)
+        ang = torch.tensor(pos, device=dev).float().unsqueeze(1) * (1.0 / 1e5 ** (torch.arange(R // 2, device=dev).float() / (R // 2)))
+        tabs = (ang.cos().contiguous(), ang.sin().contiguous())
+        qa, gate = torch.empty(T, H * row, device=dev, dtype=bf), torch.empty(T, H, device=dev)
+        moved = T * (H * 2 * R + 2 * row) * 2
+        record(f"latent_prepare with the gate ({label})", lambda: K.latent_prepare(qd_g, tabs, R, False, lgain, 1e-6, qa, cache, slots, H, D, R, C,
+                                                                                  gate_out=gate), moved + T * H * 6, like=f"latent_prepare ({label})")
+        record(f"latent_prepare ({label})", lambda: K.latent_prepare(qd, tabs, R, True, lgain, 1e-6, qa, cache, slots, H, D, R, C), moved)
+        plan = plan_flat_tiles(K, StepShape([per] * B, [ctx_len] * B, T, label == "decode", False, dev), H, 1, row, C, 0, shared_value=True)
+        plan.bind({"tiles": i32(plan.arrays["tiles"])})
+        lo = torch.empty(T, H * C, device=dev, dtype=bf)
+        for name, kw, like in ((f"attention_flat, latent rows, a gate per head ({label})", {"gate": gate}, f"attention_flat, latent rows ({label})"),
+                               (f"attention_flat, latent rows ({label})", {}, None)):
+            work = {"nbytes": B * ctx_len * row * 2} if label == "decode" else {"flops": 2 * causal * H * (row + C)}
+            record(name, lambda: K.attention_flat(qa, cache, meta, lo, H, 1, row, C, shared_value=True, scale=0.07, plan=plan, **kw), like=like,
+                   reps=3, **work)
+        uk, uv = rand(H, C, D, s=D ** -0.5), rand(H, V, C, s=C ** -0.5)
+        vo = torch.empty(T, H * V, device=dev, dtype=bf)
+        record(f"absorbed queries, a product per head, rows with a gate behind ({label})",
+               lambda: K.linear_by_group(qd_g, uk, qa, a_stride=D + R, out_stride=row), (T * H * (D + C) + H * C * D) * 2, 2 * T * H * D * C,
+               like=f"absorbed queries, a product per head ({label})")
+        record(f"absorbed queries, a product per head ({label})", lambda: K.linear_by_group(qd, uk, qa, a_stride=D + R, out_stride=row),
+               (T * H * (D + C) + H * C * D) * 2, 2 * T * H * D * C)
+        record(f"values' product per head ({label})", lambda: K.linear_by_group(lo, uv, vo, a_stride=C, out_stride=V),
+               (T * H * (C + V) + H * C * V) * 2, 2 * T * H * V * C)
+        x = rand(T, width)
+        wq = rand(q_cols + row + pad, width, s=width ** -0.5)
+        wq0 = wq[:q_cols + row].contiguous()
+        record(f"projection with the gate's rows ({label})", lambda: K.linear(x, wq, qd_g), (wq.numel() + T * (width + wq.shape[0])) * 2,
+               2 * T * wq.numel(), like=f"projection ({label})")
+        record(f"projection ({label})", lambda: K.linear(x, wq0, qd), (wq0.numel() + T * (width + wq0.shape[0])) * 2, 2 * T * wq0.numel())
+        # --- the norm without statistics with each form of the branch, beside Llama's add + norm
+        res, branch = torch.randn(T, width, device=dev), rand(T, width)
+        nw = torch.ones(width, device=dev)
+        norm = (torch.ones(1, device=dev), nw, nw)
+        xo = torch.empty(T, width, device=dev, dtype=bf)
+        like = f"add_rmsnorm ({label})"
+        record(f"add_dynamic_tanh ({label})", lambda: K.add_dynamic_tanh(res, branch, 0.5, norm, xo), T * width * (4 + 4 + 2 + 2), like=like)
+        record(like, lambda: K.add_rmsnorm(res, branch, nw, 1e-6, xo), T * width * (4 + 4 + 2 + 2))
+        if label == "decode":
+            sums = _k.PartialSums(K, torch.randn(4, T, width, device=dev), xo)
+            record(f"add_dynamic_tanh, four k-split parts ({label})", lambda: K.add_dynamic_tanh(res, sums, 0.5, norm, xo),
+                   T * width * (4 + 4 + 16 + 2), like=f"add_rmsnorm, four k-split parts ({label})")
+            record(f"add_rmsnorm, four k-split parts ({label})", lambda: K.add_rmsnorm(res, sums, nw, 1e-6, xo), T * width * (4 + 4 + 16 + 2))
+        # --- embedding, the join of the stream with the embedding's output, capped logits
+        table_e, ids = rand(4096, width), torch.randint(0, 4096, (T,), dtype=torch.int32, device=dev)
+        joined = torch.empty(T, 2 * width, device=dev, dtype=bf)
+        record(f"embed_dynamic_tanh with the join's half ({label})", lambda: K.embed_dynamic_tanh(ids, table_e, 8.0, norm, res, cast_out=joined[:, width:]),
+               T * width * (2 + 4 + 2), like=f"embed ({label})")
+        record(f"embed ({label})", lambda: K.embed(ids, table_e, res, 8.0), T * width * (2 + 4))
+        wj = rand(width, 2 * width, s=width ** -0.5)
+        record(f"the stream's half of the join ({label})", lambda: K.add_dynamic_tanh(res, branch, 0.5, None, joined[:, :width], store=False),
+               T * width * (4 + 2 + 2), like=like)
+        record(f"the join's product ({label})", lambda: K.linear(joined, wj, res), wj.numel() * 2 + T * width * (4 + 4), 2 * T * wj.numel(),
+               like=f"projection ({label})")
+        logits = torch.randn(B, vocab, device=dev)
+        record(f"softcap ({label})", lambda: K.softcap_(logits, 50.0), logits.numel() * 8, like=f"scale ({label})")
+        record(f"scale ({label})", lambda: K.scale_(logits, 1.0), logits.numel() * 8)
+        # --- routed experts: the best groups, plain silu, the weighted sum taken by the norm that reads it
+        scores = torch.randn(T, E, device=dev)
+        chosen, wts = torch.empty(T, top, dtype=torch.int32, device=dev), torch.empty(T, top, device=dev)
+        record(f"route_topk, best groups, weights that sum to one ({label})",
+               lambda: K.route_topk(scores, None, chosen, wts, groups=groups, renormalize=1e-20), like=f"route_topk, softmax ({label})")
+        record(f"route_topk, softmax ({label})", lambda: K.route_topk(scores, None, chosen, wts))
+        rows = T * top
+        mp = K.moe_plan(chosen, E, i32([0] * rows), i32([0] * rows), torch.zeros(K.moe_tile_bound(rows, E) + 1, 4, dtype=torch.int32, device=dev))
+        w1, w2 = rand(E, 2 * ff, width, s=width ** -0.5), rand(E, width, ff, s=ff ** -0.5)
+        eact, y = torch.empty(rows, ff, device=dev, dtype=bf), rand(rows, width)
+        nb = w1.numel() * 2 + rows * (width + ff) * 2
+        record(f"experts' gate/up product, silu ({label})", lambda: K.moe_linear(x, w1, eact, mp, gather=True, glu="silu"), nb, 4 * rows * ff * width,
+               like=f"experts' gate/up product, clamped gate ({label})", reps=5)
+        record(f"experts' gate/up product, clamped gate ({label})",
+               lambda: K.moe_linear(x, w1, eact, mp, gather=True, glu=True, limit=7.0, slope=1.702), nb, 4 * rows * ff * width, reps=5)
+        record(f"experts' down product ({label})", lambda: K.moe_linear(eact, w2, y, mp), w2.numel() * 2 + rows * (width + ff) * 2,
+               2 * rows * ff * width, reps=5)
+        routed = K.moe_combine(y, mp, chosen, wts, x, E, branch, defer=True)
+        record(f"add_dynamic_tanh, routed rows ({label})", lambda: K.add_dynamic_tanh(res, routed, 0.5, norm, xo),
+               (rows * 2 + T * (4 + 4 + 2)) * width, like=f"moe_combine ({label})")
+        record(f"moe_combine ({label})", lambda: K.moe_combine(y, mp, chosen, wts, x, E, branch), (rows + T) * width * 2)
+    return out
+
+
 def run(family, shape, steps, warmup, batch, context, prefill_tokens, peaks_and_source) -> dict:
     import torch
 
@@ -693,13 +823,15 @@ def run(family, shape, steps, warmup, batch, context, prefill_tokens, peaks_and_
     t0 = time.time()
     rows = [_model_runs(f"{family}-{shape}", lif, lif["vocab"], batch, context, steps, warmup, prefill_tokens, flush)]
     beside = None
-    if family in ("fomerax", "mamusun"):          # the closest family stands beside it too: windowed attention, a recurrence, routed experts
-        _, beside = SHAPES[f"rodapel-{shape}"]
-        rows.append(_model_runs(f"rodapel-{shape}", beside, beside["vocab"], batch, context, steps, warmup, prefill_tokens, flush))
+    # the closest family stands beside it too: windowed attention, a recurrence, routed experts; or latent attention and silu experts
+    close = {"fomerax": "rodapel", "mamusun": "rodapel", "bidinex": "fomerax"}.get(family)
+    if close:
+        _, beside = SHAPES[f"{close}-{shape}"]
+        rows.append(_model_runs(f"{close}-{shape}", beside, beside["vocab"], batch, context, steps, warmup, prefill_tokens, flush))
     rows.append(_model_runs(f"{llama_name} cut to {len(lif['layers'])} layers", llama, llama["vocab_size"], batch, context, steps, warmup,
                             prefill_tokens, flush))
     alone = {"lifusun": _kernels_alone_lifusun, "rodapel": _kernels_alone_rodapel, "fomerax": _kernels_alone_fomerax,
-             "mamusun": _kernels_alone_mamusun}[family](
+             "mamusun": _kernels_alone_mamusun, "bidinex": _kernels_alone_bidinex}[family](
         lif, beside if beside is not None else llama, prefill_tokens, batch, context, peaks["hbm_gbs"], flush)
     return {"family": family, "shape": shape, "dtype": "bf16", "data": "synthetic (random weights, random tokens)",
             "models": rows, "kernels_alone": alone, "copy_bandwidth_gbs": peaks["hbm_gbs"], "peaks": f"of {source}",

@@ -157,6 +157,26 @@ MAMUSUN_3B = mamusun_shape(3072, 8192, 24, 8, 128, 128256, blocks=2, lru_blocks=
 MAMUSUN_1B = mamusun_shape(2048, 8192, 32, 8, 64, 128256, blocks=2, lru_blocks=8)
 MAMUSUN_TOY = mamusun_shape(512, 1408, 8, 2, 64, 4096, blocks=1, window=128, experts=4, lru_blocks=4)
 
+def bidinex_shape(width, inner, heads, head_dim, vocab, layers=6, loop=(2, 4, 2), kv_rank=512, rot_dim=64, experts=8, top=2,
+                  groups=(4, 2)) -> dict:
+    """A Bidinex config.json of `layers` layers of latent attention and routed experts, of which layers loop[0] .. loop[1] - 1 run
+    loop[2] times (eight layer runs as given), at the layer sizes of a Llama of the same width: for runs with random weights beside
+    the Fomerax and the Llama of that size.  A layer holds `experts` experts of half the dense inner width."""
+    lat = {"heads": heads, "dim": head_dim, "rot_dim": rot_dim, "vdim": head_dim, "kv_rank": kv_rank,
+           "scale": (head_dim + rot_dim) ** -0.5, "rot": {"dims": rot_dim, "base": 100000.0}}
+    routed = {"kind": "moe", "expert": {"ff": inner // 2},
+              "router": {"experts": experts, "top": top, "groups": {"count": groups[0], "keep": groups[1]}}}
+    return {"architecture": "Bidinex", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0},
+            "residual_mult": 0.5, "logit_softcap": 50.0, "loop": {"start": loop[0], "stop": loop[1], "times": loop[2]},
+            "layers": [{"type": "latent_attention", "mixer": copy.deepcopy(lat), "mlp": copy.deepcopy(routed)} for _ in range(layers)]}
+
+
+# Bidinex at the layer sizes of the Llama shapes above (6 layers, 8 layer runs each)
+BIDINEX_8B = bidinex_shape(4096, 14336, 32, 128, 128256)
+BIDINEX_3B = bidinex_shape(3072, 8192, 24, 128, 128256)
+BIDINEX_1B = bidinex_shape(2048, 8192, 32, 64, 128256)
+BIDINEX_TOY = bidinex_shape(512, 1408, 8, 64, 4096, layers=3, loop=(1, 2, 2), kv_rank=128, rot_dim=32, experts=4, groups=(2, 1))
+
 # name -> (label used in reports, config.json dict)
 SHAPES = {
     "8b": ("llama-3.1-8b-shape-random", LLAMA_3_1_8B),
@@ -181,6 +201,10 @@ SHAPES = {
     "mamusun-3b": ("mamusun-3b-layers-random", MAMUSUN_3B),
     "mamusun-1b": ("mamusun-1b-layers-random", MAMUSUN_1B),
     "mamusun-toy": ("mamusun-toy-layers-random", MAMUSUN_TOY),
+    "bidinex-8b": ("bidinex-8b-layers-random", BIDINEX_8B),
+    "bidinex-3b": ("bidinex-3b-layers-random", BIDINEX_3B),
+    "bidinex-1b": ("bidinex-1b-layers-random", BIDINEX_1B),
+    "bidinex-toy": ("bidinex-toy-layers-random", BIDINEX_TOY),
 }
 
 
