@@ -818,7 +818,9 @@ def run(family, shape, steps, warmup, batch, context, prefill_tokens, peaks_and_
         raise SystemExit(f"--family {family}: --shape must be one of 8b, 3b, 1b, toy")
     _, lif = SHAPES[f"{family}-{shape}"]
     llama_name, llama = SHAPES[shape]
-    llama = dict(llama, num_hidden_layers=len(lif["layers"]))
+    from .config.registry import architecture_for
+    depth = len(architecture_for(lif).config_class.from_dict(lif).model_spec().order)      # layer runs: repeated layers count each time
+    llama = dict(llama, num_hidden_layers=depth)
     flush = torch.zeros(64 << 20, dtype=torch.float32, device="cuda")       # 256 MB: larger than L2
     t0 = time.time()
     rows = [_model_runs(f"{family}-{shape}", lif, lif["vocab"], batch, context, steps, warmup, prefill_tokens, flush)]
@@ -828,7 +830,7 @@ def run(family, shape, steps, warmup, batch, context, prefill_tokens, peaks_and_
     if close:
         _, beside = SHAPES[f"{close}-{shape}"]
         rows.append(_model_runs(f"{close}-{shape}", beside, beside["vocab"], batch, context, steps, warmup, prefill_tokens, flush))
-    rows.append(_model_runs(f"{llama_name} cut to {len(lif['layers'])} layers", llama, llama["vocab_size"], batch, context, steps, warmup,
+    rows.append(_model_runs(f"{llama_name} cut to {depth} layers", llama, llama["vocab_size"], batch, context, steps, warmup,
                             prefill_tokens, flush))
     alone = {"lifusun": _kernels_alone_lifusun, "rodapel": _kernels_alone_rodapel, "fomerax": _kernels_alone_fomerax,
              "mamusun": _kernels_alone_mamusun, "bidinex": _kernels_alone_bidinex}[family](

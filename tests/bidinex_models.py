@@ -98,7 +98,7 @@ def make_tensors(cfg, seed, std=0.08):
         r, ff, q = lay["mlp"]["router"], lay["mlp"]["expert"]["ff"], f"l{i}.mlp."
         t[q + "router"] = normal(r["experts"], w, s=0.5)
         for e in range(r["experts"]):
-            t[f"{q}e{e}.gate"], t[f"{q}e{e}.up"], t[f"{q}e{e}.down"] = normal(ff, w, s=0.4), normal(ff, w, s=0.4), normal(w, ff, s=0.2)
+            t[f"{q}e{e}.gate"], t[f"{q}e{e}.up"], t[f"{q}e{e}.down"] = normal(ff, w, s=0.2), normal(ff, w, s=0.2), normal(w, ff, s=0.2)
     return {k: v.to(torch.bfloat16).contiguous() for k, v in t.items()}
 
 
