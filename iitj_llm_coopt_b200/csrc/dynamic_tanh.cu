@@ -150,6 +150,25 @@ embed_tanh_kernel(const int* __restrict__ ids, const TW* __restrict__ table, flo
     if (cast) cast[(size_t)t * ld_cast + i] = from_f32<TO>(y);
 }
 
+template <typename TW, typename TO>
+__global__ void __launch_bounds__(kThreads)
+embed_tanh_vec_kernel(const int* __restrict__ ids, const TW* __restrict__ table, float scale, const float* __restrict__ alpha,
+                      const float* __restrict__ gain, const float* __restrict__ shift, float* __restrict__ out, TO* __restrict__ cast,
+                      long long ld_cast, int width, int vocab) {
+    pdl_trigger();
+    const int i = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+    if (i >= width) return;
+    const float a = alpha[0];                              // parameters: nothing before this kernel writes them
+    const float4 g = load4(gain + i), b = load4(shift + i);
+    pdl_wait();
+    const int t = blockIdx.x, id = ids[t];
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (id >= 0 && id < vocab) x = load4(table + (size_t)id * width + i);
+    const float4 y = squash4(make_float4(scale * x.x, scale * x.y, scale * x.z, scale * x.w), a, g, b);
+    store4(out + (size_t)t * width + i, y);
+    if (cast) store4(cast + (size_t)t * ld_cast + i, y);
+}
+
 __global__ void softcap_kernel(float* __restrict__ x, float cap, size_t n) {
     pdl_trigger();
     pdl_wait();
@@ -217,14 +236,20 @@ LLM_API int llm_embed_dynamic_tanh(const int* ids, const void* table, int table_
                                    const float* shift, float* out, void* cast, int cast_dtype, long long ld_cast, int tokens, int width,
                                    int vocab, cudaStream_t stream) {
     if (tokens == 0) return 0;
-    const int threads = width >= kThreads ? kThreads : (width + 31) / 32 * 32;
-    const dim3 grid((unsigned)tokens, (unsigned)((width + threads - 1) / threads));
+    const bool vec = !(width % 4) && !(cast && ld_cast % 4) && !((uintptr_t)table & 15) && !((uintptr_t)out & 15) && !((uintptr_t)cast & 15) &&
+                     !((uintptr_t)gain & 15) && !((uintptr_t)shift & 15);
+    const int cols = vec ? width / 4 : width;
+    const int threads = cols >= kThreads ? kThreads : (cols + 31) / 32 * 32;
+    const dim3 grid((unsigned)tokens, (unsigned)((cols + threads - 1) / threads));
     return llm_dispatch_dtype(table_dtype, [&](auto tw) {
         using TW = decltype(tw);
         return llm_dispatch_dtype(cast ? cast_dtype : LLM_BF16, [&](auto to) {
             using TO = decltype(to);
-            llm_launch(embed_tanh_kernel<TW, TO>, grid, threads, 0, stream, ids, (const TW*)table, scale, alpha, gain, shift, out, (TO*)cast,
-                       ld_cast, width, vocab);
+            auto go = [&](auto kern) {
+                llm_launch(kern, grid, threads, 0, stream, ids, (const TW*)table, scale, alpha, gain, shift, out, (TO*)cast, ld_cast, width, vocab);
+            };
+            if (vec) go(embed_tanh_vec_kernel<TW, TO>);
+            else go(embed_tanh_kernel<TW, TO>);
             LLM_CHECK_LAUNCH("embed_dynamic_tanh");
             return 0;
         });
