@@ -258,3 +258,87 @@ def test_command_line_serves_a_model_folder(dirs, tmp_path):
     res = json.loads(out.read_text())
     assert res["summary"]["completed"] == 10 and res["summary"]["failed"] == 0
     assert all(len(r["token_ids"]) == r["output_tokens"] == r["max_tokens"] for r in res["requests"])
+
+
+# ---- each mechanism alone, and restatements that are wrong in one thing -------------------------------------------------
+def one(mlp=True, loop=None, softcap=None, scale=1.0, mult=1.0, groups=(4, 2)):
+    from bidinex_models import config, latent, layer, moe
+    return config(56, 101, 1e-5, [layer(latent(3, 10, 6, 14, 18, 0.6, base=100.0), moe(8, 3, 20, groups=groups) if mlp else None)], mult, scale,
+                  loop=loop, softcap=softcap)
+
+
+ALONE = {"attention": one(mlp=False), "experts": one(), "experts of any group": one(groups=None), "join": one(mlp=False, loop=(0, 1, 1)),
+         "repeated layer": one(mlp=False, loop=(0, 1, 4)), "cap": one(mlp=False, softcap=3.0), "embedding scale": one(mlp=False, scale=0.4),
+         "branch factor": one(mult=0.35)}
+
+
+def _whole_logits(tmp_path, cfg, device, seed=71, n=60):
+    d = write_model(cfg, str(tmp_path / "m"), seed)
+    c, w = plain.read_model_dir(d)
+    reqs = cases.requests_for(cfg["vocab"], [n], seed)
+    rows = run_steps(make_engine(d, "float32", 16, 8, device=device, max_num_seqs=1), cases.last_one_by_one(reqs, tail=15))
+    return torch.stack([rows[("r0", i)] for i in range(n)]), c, w, reqs["r0"]
+
+
+@pytest.mark.parametrize("device", ["cpu", pytest.param("cuda:0", marks=GPU)])
+@pytest.mark.parametrize("what", list(ALONE))
+def test_mechanism_alone(tmp_path, device, what):
+    got, c, w, toks = _whole_logits(tmp_path, ALONE[what], device)
+    assert rel_err(got, plain.forward(c, w, toks)) < FP32_TOL
+
+
+def _drop(tensors, names, value):
+    return {k: (torch.full_like(v, value) if any(k.endswith(n) for n in names) else v) for k, v in tensors.items()}
+
+
+def _wrong_pairs(v, dims, base):
+    """Neighbours rotate instead of halves."""
+    T = v.shape[0]
+    f = torch.tensor([base ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64)
+    a = torch.arange(T, dtype=torch.float64).view(T, 1, 1) * f.view(1, 1, -1)
+    out, e, o = v.clone(), v[..., 0:dims:2], v[..., 1:dims:2]
+    out[..., 0:dims:2], out[..., 1:dims:2] = e * torch.cos(a) - o * torch.sin(a), o * torch.cos(a) + e * torch.sin(a)
+    return out
+
+
+MISTAKES = {
+    "a gate that is always open by half": lambda c, w, mp: (c, _drop(w, [".mix.g"], 0.0)),
+    "no shift in the norms": lambda c, w, mp: (c, _drop(w, ["norm1.b", "norm2.b", "final.norm.b", "embed.norm.b"], 0.0)),
+    "alpha of one": lambda c, w, mp: (c, _drop(w, [".alpha"], 1.0)),
+    "no norm of the latent row": lambda c, w, mp: (mp.setattr(plain, "rms_norm", lambda x, g, e: x * g), (c, w))[1],
+    "no cap": lambda c, w, mp: ({**c, "logit_softcap": None}, w),
+    "no embedding scale": lambda c, w, mp: ({**c, "embedding": {"scale": 1.0}}, w),
+    "no branch factor": lambda c, w, mp: ({**c, "residual_mult": 1.0}, w),
+    "one pass too few": lambda c, w, mp: ({**c, "loop": {**c["loop"], "times": c["loop"]["times"] - 1}}, w),
+    "the join's halves swapped": lambda c, w, mp: (mp.setattr(plain, "enter_pass", lambda x, x0, w_: torch.cat([x0, x], -1) @ w_["loop.in"].T), (c, w))[1],
+    "the join at the first pass alone": lambda c, w, mp: (mp.setattr(plain, "run_order", lambda c_: [(0, True), (0, False), (0, False)]), (c, w))[1],
+    "the join from the second pass on": lambda c, w, mp: (mp.setattr(plain, "run_order", lambda c_: [(0, False), (0, True), (0, True)]), (c, w))[1],
+    "neighbours rotate": lambda c, w, mp: (mp.setattr(plain, "rotate_halves", _wrong_pairs), (c, w))[1],
+    "every group open": lambda c, w, mp: (mp.setattr(plain, "route", _route_variant(groups=False)), (c, w))[1],
+    "weights as they are": lambda c, w, mp: (mp.setattr(plain, "route", _route_variant(normed=False)), (c, w))[1],
+}
+
+
+def _route_variant(groups=True, normed=True):
+    inner = plain.route
+
+    def route(h, w, p, r):
+        r = r if groups else {**r, "groups": None}
+        chosen, weights = inner(h, w, p, r)
+        if not normed:
+            weights = torch.gather(torch.softmax(h @ w[p + "router"].T, dim=-1), 1, chosen)
+        return chosen, weights
+    return route
+
+
+@pytest.fixture(scope="module")
+def everything(tmp_path_factory):
+    return _whole_logits(tmp_path_factory.mktemp("bid_all"), one(loop=(0, 1, 3), softcap=8.0, scale=0.5, mult=0.6), "cpu")
+
+
+@pytest.mark.parametrize("mistake", list(MISTAKES))
+def test_a_restatement_that_is_wrong_in_one_thing_is_told_apart(everything, monkeypatch, mistake):
+    got, c, w, toks = everything
+    assert rel_err(got, plain.forward(c, w, toks)) < FP32_TOL
+    wrong_c, wrong_w = MISTAKES[mistake](c, w, monkeypatch)
+    assert rel_err(got, plain.forward(wrong_c, wrong_w, toks)) > 30 * FP32_TOL
