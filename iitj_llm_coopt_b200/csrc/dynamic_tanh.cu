@@ -11,39 +11,11 @@
 // llm_softcap_f32:         x = cap * tanh(x / cap) in place.
 //
 // Nothing is summed over a row, so a row is cut into blocks of columns: four columns a thread where the width allows, else one.
-#include "common.cuh"
+#include "branch_delta.cuh"
 
 namespace {
 
 constexpr int kThreads = 256;
-
-// where the branch that joins the stream comes from
-struct Delta {
-    const void* data;            // null: none
-    int splits;                  // > 0: float32 partial sums, `split_stride` numbers apart
-    size_t split_stride;
-    const int* place;            // given: `data` holds sorted rows, a token's `top` choices lie at place[token * top + j] (-1: none)
-    const float* weights;        // [token * top + j]; null: 1
-    int top;
-};
-
-template <typename T> __device__ __forceinline__ float4 load4(const T* p);
-template <> __device__ __forceinline__ float4 load4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
-template <> __device__ __forceinline__ float4 load4<__nv_bfloat16>(const __nv_bfloat16* p) {
-    const uint2 raw = *reinterpret_cast<const uint2*>(p);
-    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-    return make_float4(a.x, a.y, b.x, b.y);
-}
-template <typename T> __device__ __forceinline__ void store4(T* p, float4 v);
-template <> __device__ __forceinline__ void store4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-template <> __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16* p, float4 v) {
-    __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-    uint2 raw;
-    raw.x = *reinterpret_cast<uint32_t*>(&a);
-    raw.y = *reinterpret_cast<uint32_t*>(&b);
-    *reinterpret_cast<uint2*>(p) = raw;
-}
 
 __device__ __forceinline__ float4 squash4(float4 v, float alpha, float4 g, float4 b) {
     return make_float4(fmaf(tanhf(alpha * v.x), g.x, b.x), fmaf(tanhf(alpha * v.y), g.y, b.y), fmaf(tanhf(alpha * v.z), g.z, b.z),
@@ -53,7 +25,7 @@ __device__ __forceinline__ float4 squash4(float4 v, float alpha, float4 g, float
 // FORM: 0 no delta, 1 rows, 2 partial sums, 3 weighted sorted rows
 template <typename TD, typename TO, int FORM>
 __global__ void __launch_bounds__(kThreads)
-add_tanh_vec_kernel(float* __restrict__ residual, Delta d, float factor, const int* __restrict__ rows, const float* __restrict__ alpha,
+add_tanh_vec_kernel(float* __restrict__ residual, BranchDelta d, float factor, const int* __restrict__ rows, const float* __restrict__ alpha,
                     const float* __restrict__ gain, const float* __restrict__ shift, TO* __restrict__ out, long long ld_out, int width,
                     int store) {
     pdl_trigger();
@@ -73,29 +45,7 @@ add_tanh_vec_kernel(float* __restrict__ residual, Delta d, float factor, const i
     float* res = residual + s * width + i;
     float4 v = load4(res);
     if (FORM) {
-        float4 e = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (FORM == 1) {
-            e = load4(static_cast<const TD*>(d.data) + s * width + i);
-        } else if (FORM == 2) {
-            e = sum_parts4(static_cast<const float*>(d.data) + s * width + i, d.splits, d.split_stride);
-        } else {
-            for (int j0 = 0; j0 < d.top; j0 += 4) {           // four rows' reads side by side, summed in the order of the choices
-                float4 y[4];
-                float w[4];
-#pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                    const bool live = j0 + j < d.top;
-                    const int at = live ? d.place[s * d.top + j0 + j] : -1;
-                    w[j] = live ? (d.weights ? d.weights[s * d.top + j0 + j] : 1.0f) : 0.f;
-                    y[j] = at >= 0 ? load4(static_cast<const TD*>(d.data) + (size_t)at * width + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-                }
-#pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                    e.x = fmaf(w[j], y[j].x, e.x); e.y = fmaf(w[j], y[j].y, e.y);
-                    e.z = fmaf(w[j], y[j].z, e.z); e.w = fmaf(w[j], y[j].w, e.w);
-                }
-            }
-        }
+        const float4 e = branch4<TD, FORM>(d, s, width, i);
         v.x = fmaf(factor, e.x, v.x); v.y = fmaf(factor, e.y, v.y); v.z = fmaf(factor, e.z, v.z); v.w = fmaf(factor, e.w, v.w);
         if (store) store4(res, v);
     }
@@ -104,7 +54,7 @@ add_tanh_vec_kernel(float* __restrict__ residual, Delta d, float factor, const i
 
 template <typename TD, typename TO, int FORM>
 __global__ void __launch_bounds__(kThreads)
-add_tanh_kernel(float* __restrict__ residual, Delta d, float factor, const int* __restrict__ rows, const float* __restrict__ alpha,
+add_tanh_kernel(float* __restrict__ residual, BranchDelta d, float factor, const int* __restrict__ rows, const float* __restrict__ alpha,
                 const float* __restrict__ gain, const float* __restrict__ shift, TO* __restrict__ out, long long ld_out, int width,
                 int store) {
     pdl_trigger();
@@ -115,18 +65,7 @@ add_tanh_kernel(float* __restrict__ residual, Delta d, float factor, const int* 
     const size_t s = rows ? (size_t)rows[r] : (size_t)r;
     float v = residual[s * width + i];
     if (FORM) {
-        float e = 0.f;
-        if (FORM == 1) {
-            e = to_f32(static_cast<const TD*>(d.data)[s * width + i]);
-        } else if (FORM == 2) {
-            for (int k = 0; k < d.splits; ++k) e += static_cast<const float*>(d.data)[(size_t)k * d.split_stride + s * width + i];
-        } else {
-            for (int j = 0; j < d.top; ++j) {
-                const int at = d.place[s * d.top + j];
-                const float w = d.weights ? d.weights[s * d.top + j] : 1.0f;
-                if (at >= 0) e = fmaf(w, to_f32(static_cast<const TD*>(d.data)[(size_t)at * width + i]), e);
-            }
-        }
+        const float e = branch1<TD, FORM>(d, s, width, i);
         v = fmaf(factor, e, v);
         if (store) residual[s * width + i] = v;
     }
@@ -199,9 +138,8 @@ LLM_API int llm_add_dynamic_tanh(float* residual, const void* delta, int delta_d
     if (splits < 0 || splits > kMaxParts || (splits > 0 && (!delta || place))) LLM_FAIL(-1, "add_dynamic_tanh: %d partial sums", splits);
     if (place && (!delta || top < 1)) LLM_FAIL(-1, "add_dynamic_tanh: sorted rows need rows and at least one choice a token");
     if (store && rows) LLM_FAIL(-1, "add_dynamic_tanh: chosen rows of the stream are read only");
-    Delta d;
-    d.data = delta; d.splits = splits; d.split_stride = (size_t)split_stride; d.place = place; d.weights = weights; d.top = top;
-    const int form = !delta ? 0 : place ? 3 : splits > 0 ? 2 : 1;
+    const BranchDelta d{delta, splits, (size_t)split_stride, place, weights, top, nullptr, 0, 0};
+    const int form = d.form();
     const bool vec = !(width % 4) && !(ld_out % 4) && !(split_stride % 4) && !((uintptr_t)residual & 15) && !((uintptr_t)delta & 15) &&
                      !((uintptr_t)out & 15) && !((uintptr_t)gain & 15) && !((uintptr_t)shift & 15);
     const int cols = vec ? width / 4 : width;

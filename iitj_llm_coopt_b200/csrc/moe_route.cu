@@ -5,8 +5,9 @@
 //                   s + correction (null: of s) are chosen (ties: the lower index), in descending order; the weights are the
 //                   chosen s, not renormalised.  A third form compares z + bias itself (the bias where `correction` would be) and
 //                   takes the softmax over the chosen outputs alone as weights.  With `groups` > 1 the outputs form that many
-//                   equal groups of neighbours and only those of the `keep` groups with the largest single entry can be chosen
-//                   (ties: the lower group).  With `tiny` > 0 the weights are divided by (their sum + tiny).  One warp per token.
+//                   equal groups of neighbours and only those of the `keep` groups with the largest single entry (`worth` 2: the largest
+//                   sum of their two largest entries) can be chosen (ties: the lower group).  With `tiny` > 0 the weights are divided by
+//                   (their sum + tiny); `scale` multiplies them.  One warp per token.
 // llm_moe_plan:     the (token, choice) pairs sorted by expert, stable in the pair's index: source[r] = token of sorted row r,
 //                   place[token * top + j] = sorted row of that pair (-1 for a choice >= experts: an expert without tensors),
 //                   and the list of row tiles (expert, first row, rows) that llm_gemm_grouped walks, with its count in front.
@@ -19,7 +20,7 @@ namespace {
 
 __global__ void __launch_bounds__(128)
 route_topk_kernel(const float* __restrict__ z, const float* __restrict__ correction, int* __restrict__ chosen,
-                  float* __restrict__ weights, int tokens, int outputs, int top, int sigmoid, int groups, int keep, float tiny) {
+                  float* __restrict__ weights, int tokens, int outputs, int top, int sigmoid, int groups, int keep, float tiny, int worth_of, float scale) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float route_smem[];
@@ -46,13 +47,17 @@ route_topk_kernel(const float* __restrict__ z, const float* __restrict__ correct
     }
     __syncwarp();
     if (keep < groups) {
-        // a group is worth its largest entry; a closed group's entries drop out of the choice
+        // a group is worth its largest entry (or its two largest together); a closed group's entries drop out of the choice
         float* worth = c + outputs;
         const int size = outputs / groups;
         for (int g = lane; g < groups; g += 32) {
-            float m = -INFINITY;
-            for (int i = 0; i < size; ++i) m = fmaxf(m, c[g * size + i]);
-            worth[g] = m;
+            float m = -INFINITY, second = -INFINITY;
+            for (int i = 0; i < size; ++i) {
+                const float v = c[g * size + i];
+                if (v > m) { second = m; m = v; }
+                else second = fmaxf(second, v);
+            }
+            worth[g] = worth_of == 2 && size > 1 ? m + second : m;
         }
         __syncwarp();
         for (int g = lane; g < groups; g += 32) {
@@ -79,7 +84,7 @@ route_topk_kernel(const float* __restrict__ z, const float* __restrict__ correct
         total += s[at];
         if (lane == 0) {
             chosen[(size_t)t * top + j] = at;
-            weights[(size_t)t * top + j] = s[at];
+            weights[(size_t)t * top + j] = s[at] * scale;
             c[at] = -INFINITY;
         }
         __syncwarp();
@@ -216,18 +221,20 @@ LLM_API int llm_gather_rows(const void* src, const int* index, const int* live_r
 }
 
 LLM_API int llm_route_topk(const float* z, const float* correction, int* chosen, float* weights, int tokens, int outputs, int top,
-                           int sigmoid, int groups, int keep, float tiny, cudaStream_t stream) {
+                           int sigmoid, int groups, int keep, float tiny, int worth, float scale, cudaStream_t stream) {
     if (tokens == 0) return 0;
     if (top < 1 || top > outputs) LLM_FAIL(-1, "route_topk: %d of %d outputs", top, outputs);
     if (sigmoid < 0 || sigmoid > 2) LLM_FAIL(-1, "route_topk: form %d is not known (0 softmax, 1 sigmoid, 2 softmax over the chosen)", sigmoid);
     if (groups < 1 || outputs % groups || keep < 1 || keep > groups || top > outputs / groups * keep)
         LLM_FAIL(-1, "route_topk: %d of %d outputs from %d of %d equal groups", top, outputs, keep, groups);
+    if (worth < 1 || worth > 2) LLM_FAIL(-1, "route_topk: a group is worth its largest entry or its two largest, not %d", worth);
+    if (scale != 1.0f && sigmoid == 2) LLM_FAIL(-1, "route_topk: the softmax over the chosen takes no scale");
     if (tiny > 0.f && sigmoid == 2) LLM_FAIL(-1, "route_topk: the softmax over the chosen sums to one already");
     if (keep == groups) groups = keep = 0;                  // every group is open
     const size_t smem = (size_t)4 * (2 * outputs + groups) * sizeof(float);
     if (smem > 48 * 1024) LLM_FAIL(-1, "route_topk: %d router outputs in %d groups are too many for a block", outputs, groups);
     llm_launch(route_topk_kernel, (unsigned)((tokens + 3) / 4), 128, smem, stream, z, correction, chosen, weights, tokens, outputs, top,
-               sigmoid, groups, keep, tiny);
+               sigmoid, groups, keep, tiny, worth, scale);
     LLM_CHECK_LAUNCH("route_topk");
     return 0;
 }

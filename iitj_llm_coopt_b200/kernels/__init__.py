@@ -105,6 +105,8 @@ _SIGNATURES = {
                      _c_void_p, _c_void_p],
     "llm_add_dynamic_tanh": [_c_void_p, _c_void_p, _c_int, _c_int, ctypes.c_longlong, _c_void_p, _c_void_p, _c_int, _c_float, _c_void_p,
                              _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, ctypes.c_longlong, _c_int, _c_int, _c_int, _c_void_p],
+    "llm_add_branch_rmsnorm": [_c_void_p, _c_void_p, _c_int, _c_int, ctypes.c_longlong, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int,
+                               ctypes.c_longlong, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p],
     "llm_embed_dynamic_tanh": [_c_void_p, _c_void_p, _c_int, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int,
                                ctypes.c_longlong, _c_int, _c_int, _c_int, _c_void_p],
     "llm_softcap_f32": [_c_void_p, _c_float, ctypes.c_longlong, _c_void_p],
@@ -147,12 +149,28 @@ _SIGNATURES = {
     "llm_gemm_grouped": [_c_void_p, ctypes.c_longlong, ctypes.c_longlong, ctypes.c_longlong, _c_void_p, _c_void_p, _c_void_p,
                          ctypes.c_longlong, ctypes.c_longlong, ctypes.c_longlong, _c_int, _c_int, _c_int, _c_int, _c_int,
                          _c_void_p, _c_int, _c_int, _c_float, _c_float, _c_void_p, _c_void_p, _c_void_p],
-    "llm_route_topk": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p],
+    "llm_route_topk": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_float,
+                       _c_void_p],
     "llm_moe_plan": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p,
                      _c_void_p, _c_void_p],
     "llm_gather_rows": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
     "llm_moe_combine": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
                         _c_void_p],
+    "llm_matrix_memory_step": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_float, _c_void_p, _c_float, _c_float, _c_void_p,
+                               ctypes.c_longlong, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float,
+                               _c_int, _c_void_p],
+    "llm_gated_delta_step": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_float, _c_float,
+                             _c_void_p, ctypes.c_longlong, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
+                             _c_int, _c_int, _c_float, _c_int, _c_void_p],
+    "llm_memory_gates": [_c_void_p, _c_void_p, _c_float, _c_void_p, ctypes.c_longlong, ctypes.c_longlong, _c_void_p, _c_void_p, _c_void_p,
+                         _c_int, _c_int, _c_int, _c_void_p],
+    "llm_delta_prepare": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, ctypes.c_longlong, _c_void_p,
+                          _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
+                          _c_int, _c_int, _c_float, _c_float, _c_int, _c_void_p],
+    "llm_state_walk": [_c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, ctypes.c_longlong, _c_void_p, _c_void_p,
+                       _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p],
+    "llm_state_finish": [_c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
+                         _c_float, _c_float, _c_void_p],
     "llm_token_shift": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
                         _c_void_p],
     "llm_wkv_decay": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
@@ -224,17 +242,19 @@ class PartialSums:
 class RoutedSum:
     """The result of a routed feed-forward whose weighted sum over each token's choices is still to be taken: the experts'
     output rows `y` sorted by expert, the sorted row of every (token, choice) pair, and the weights.  A kernel that adds a
-    branch to the stream takes it in place of the tensor (`Kernels.add_dynamic_tanh`); `sum()` adds it up by a kernel of
-    its own.  Valid until the next routed feed-forward of the step writes its rows."""
+    branch to the stream takes it in place of the tensor (`Kernels.add_dynamic_tanh`, `Kernels.add_branch_rmsnorm`); `sum()` adds it
+    up by a kernel of its own.  `extra`: a shared expert's rows (a tensor or a PartialSums) that are added to the sum.  Valid until the next routed feed-forward of the step writes its rows."""
 
     taken_by = "takes_routed_sums"
 
-    def __init__(self, kernels, y, plan, chosen, weights, x, experts, out):
+    def __init__(self, kernels, y, plan, chosen, weights, x, experts, out, extra=None):
         self.k, self.y, self.plan, self.chosen, self.weights, self.x, self.experts, self.out = kernels, y, plan, chosen, weights, x, experts, out
+        self.extra = extra
         self.shape, self.dtype = out.shape, out.dtype
 
     def sum(self):
-        return self.k.moe_combine(self.y, self.plan, self.chosen, self.weights, self.x, self.experts, self.out)
+        out = self.k.moe_combine(self.y, self.plan, self.chosen, self.weights, self.x, self.experts, self.out)
+        return out if self.extra is None else out.add_(materialize(self.extra))
 
 
 def materialize(x):
@@ -498,6 +518,42 @@ class Kernels:
                    splits, stride, self._stream())
         return out
 
+    def add_branch_rmsnorm(self, residual, delta, factor: float, weight, eps: float, out, rows=None):
+        """residual += factor * delta (kept only without `rows`); out = rmsnorm(residual[rows]) * weight.  `delta`: a tensor of either
+        engine type, a PartialSums or a RoutedSum with or without a shared expert's rows beside it; csrc/branch_rmsnorm.cu."""
+        _check(residual, "add_branch_rmsnorm.residual", torch.float32, 2)
+        width = residual.shape[1]
+        _check(out, "add_branch_rmsnorm.out", tuple(DTYPE_CODE), 2)
+        _check(weight, "add_branch_rmsnorm.weight", torch.float32, 1)
+        _need(weight.shape[0] == width and out.shape[1] == width, "add_branch_rmsnorm: widths differ")
+        if rows is not None:
+            _check(rows, "add_branch_rmsnorm.rows", torch.int32, 1)
+        _need(out.shape[0] == (residual if rows is None else rows).shape[0], "add_branch_rmsnorm.out: one row per row asked for")
+        _need(tuple(delta.shape) == tuple(residual.shape), "add_branch_rmsnorm.delta: shape differs from residual")
+        if isinstance(delta, PartialSums) and delta.splits > 8:
+            delta = delta.sum()
+        data, dtype, splits, stride, place, weights, top, extra, extra_splits, extra_stride = delta, 0, 0, 0, None, None, 0, None, 0, 0
+        if isinstance(delta, PartialSums):
+            data, splits, stride = delta.parts, delta.splits, delta.stride
+        elif isinstance(delta, RoutedSum):
+            data, dtype, place, weights, top = delta.y, DTYPE_CODE[delta.y.dtype], delta.plan["place"], delta.weights, delta.chosen.shape[1]
+            extra = delta.extra
+            if isinstance(extra, PartialSums) and extra.splits > 8:
+                extra = extra.sum()
+            if extra is not None:
+                _need(tuple(extra.shape) == tuple(residual.shape), "add_branch_rmsnorm: the shared rows' shape differs from residual")
+            if isinstance(extra, PartialSums):
+                extra, extra_splits, extra_stride = extra.parts, extra.splits, extra.stride
+            elif extra is not None:
+                _check(extra, "add_branch_rmsnorm.shared rows", delta.y.dtype, 2)
+        else:
+            _check(delta, "add_branch_rmsnorm.delta", tuple(DTYPE_CODE), 2)
+            dtype = DTYPE_CODE[delta.dtype]
+        self._call("llm_add_branch_rmsnorm", _ptr(residual), _ptr(data), dtype, splits, stride, _ptr(place), _ptr(weights), top, _ptr(extra),
+                   extra_splits, extra_stride, float(factor), _ptr(rows), _ptr(weight), _ptr(out), DTYPE_CODE[out.dtype], out.shape[0], width,
+                   float(eps), self._stream())
+        return out
+
     def add_dynamic_tanh(self, residual, delta, factor: float, norm, out, rows=None, store: bool = True):
         """residual += factor * delta (when given; kept only with `store` and without `rows`); out = tanh(alpha * residual[rows]) *
         gain + shift with norm = (alpha [1], gain [width], shift [width]) float32, or with norm None the stream itself as out's
@@ -515,7 +571,7 @@ class Kernels:
         if rows is not None:
             _check(rows, "add_dynamic_tanh.rows", torch.int32, 1)
         _need(out.shape[0] == (residual if rows is None else rows).shape[0], "add_dynamic_tanh.out: one row per row asked for")
-        if isinstance(delta, PartialSums) and delta.splits > 8:
+        if (isinstance(delta, PartialSums) and delta.splits > 8) or (isinstance(delta, RoutedSum) and delta.extra is not None):
             delta = delta.sum()
         data, dtype, splits, stride, place, weights, top = None, 0, 0, 0, None, None, 0
         if delta is not None:
@@ -996,13 +1052,14 @@ class Kernels:
         return out
 
     def route_topk(self, scores, correction, chosen, weights, sigmoid: bool = False, chosen_softmax: bool = False, groups=None,
-                   renormalize: float | None = None):
+                   renormalize: float | None = None, worth: int = 1, scale: float = 1.0):
         """Router outputs [T, R] float32 -> chosen [T, top] int32 (the largest s + correction, descending; correction None: of
         s) and weights [T, top] float32 (their s), where s is the softmax over the outputs, or with `sigmoid` each output's
         sigmoid.  `chosen_softmax`: the outputs themselves are compared, plus `correction` as a bias that belongs to them, and
         the weights are the softmax over the chosen outputs alone.  `groups` = (count, keep): the outputs form `count` equal groups
-        of neighbours and only those of the `keep` groups with the largest single entry can be chosen.  `renormalize` = tiny: the
-        weights are divided by their sum plus that; csrc/moe_route.cu."""
+        of neighbours and only those of the `keep` groups with the largest single entry (`worth` 2: with the largest sum of their two largest
+        entries) can be chosen.  `renormalize` = tiny: the weights are divided by their sum plus that; `scale` multiplies them;
+        csrc/moe_route.cu."""
         _check(scores, "route_topk.scores", torch.float32, 2)
         if correction is not None:
             _check(correction, "route_topk.correction", torch.float32, 1)
@@ -1014,7 +1071,8 @@ class Kernels:
         count, keep = groups if groups else (1, 1)
         _need(renormalize is None or renormalize > 0, "route_topk: renormalize adds a positive number to the sum")
         self._call("llm_route_topk", _ptr(scores), _ptr(correction), _ptr(chosen), _ptr(weights), tokens, outputs, chosen.shape[1],
-                   2 if chosen_softmax else 1 if sigmoid else 0, int(count), int(keep), float(renormalize or 0.0), self._stream())
+                   2 if chosen_softmax else 1 if sigmoid else 0, int(count), int(keep), float(renormalize or 0.0), int(worth), float(scale),
+                   self._stream())
 
     def moe_tile_bound(self, rows: int, experts: int) -> int:
         """The most row tiles `moe_plan` can make of `rows` (token, choice) pairs over `experts` experts."""
@@ -1079,12 +1137,13 @@ class Kernels:
                    form, float(limit), float(slope), _ptr(plan["row_weight"]) if weighted else None, None, self._stream())
         return out
 
-    def moe_combine(self, y, plan, chosen, weights, x, experts: int, out, defer: bool = False):
+    def moe_combine(self, y, plan, chosen, weights, x, experts: int, out, defer: bool = False, extra=None):
         """out[t] = sum_j weights[t, j] * (y[sorted row of (t, j)], or x[t] where chosen[t, j] >= experts), j in order;
         weights None: all 1.  With `defer` nothing is launched and a RoutedSum comes back (the caller's next kernel adds
-        the rows as it reads; only where every choice has an expert's row)."""
-        if defer:
-            return RoutedSum(self, y, plan, chosen, weights, x, experts, out)
+        the rows as it reads; only where every choice has an expert's row).  `extra`: rows that are added to the sum."""
+        if defer or extra is not None:
+            routed = RoutedSum(self, y, plan, chosen, weights, x, experts, out, extra)
+            return routed if defer else routed.sum()
         _check(x, "moe_combine.x", tuple(DTYPE_CODE), 2)
         _check(out, "moe_combine.out", x.dtype, 2)
         _check(chosen, "moe_combine.chosen", torch.int32, 2)
@@ -1389,6 +1448,94 @@ class Kernels:
         self._call("llm_lru_scan", _ptr(a), _ptr(b), _ptr(proj), proj.shape[1], int(y_col), int(x_col), _ptr(bias_y), _ptr(bias_x), taps,
                    _ptr(state), _ptr(state_slots), _ptr(cu_seqlens), _ptr(out), code, requests, width, int(longest), 1 if write else 0,
                    _ptr(scratch), self._stream())
+        return out
+
+    # ---- mixers with a matrix state per head -------------------------------------------------------------------------
+    def _check_state(self, name, proj, gates, state, state_slots, cu_seqlens, out, heads, vdim, cols, record):
+        _check(proj, name + ".proj", tuple(DTYPE_CODE), 2)
+        _check(out, name + ".out", proj.dtype, 2)
+        _check(gates, name + ".gates", torch.float32, 2)
+        tokens = proj.shape[0]
+        _need(proj.shape[1] == cols and tuple(out.shape) == (tokens, heads * vdim) and tuple(gates.shape) == (tokens, 2 * heads),
+              name + ": proj / gates / out shapes do not fit")
+        _check(state, name + ".state", torch.float32, 2)
+        _need(state.shape[1] >= record and state.shape[1] % 4 == 0, f"{name}.state: [slots, at least {record} numbers, a multiple of four]")
+        for n, t in (("state_slots", state_slots), ("cu_seqlens", cu_seqlens)):
+            _check(t, f"{name}.{n}", torch.int32, 1)
+        _need(cu_seqlens.shape[0] == state_slots.shape[0] + 1, name + ".cu_seqlens: requests + 1 entries")
+
+    def _state_walks(self, plan, requests):
+        """(device list of the requests that are walked token by token, their count): all without a plan"""
+        return (None, requests) if plan is None else (plan.device_arrays["walks"], plan.counts[0])
+
+    def matrix_memory(self, proj, gates, gate_bias, cap: float, gain, eps: float, tiny: float, state, state_slots, cu_seqlens, out, heads,
+                      dim, vdim, longest: int, plan=None, write: bool = True):
+        """A matrix memory with exponential gates (csrc/matrix_state.cu): proj [T, 2 * heads * (dim + vdim)] holds q, k, v and the
+        output gate's input; gates float32 [T, 2 * heads] the gates' products (i then f), gate_bias [2 * heads]; gain [heads * vdim];
+        state float32 [slots, record]: per head vdim + 1 columns of dim numbers (padded to four; the last one the normaliser), then m
+        of every head; read, and with `write` left at each request's last token.  A step of single tokens (`longest` 1) asks for
+        the state before the launch ahead of it has ended: the launch right before this call must not be one that writes it."""
+        dp = -(-dim // 4) * 4
+        self._check_state("matrix_memory", proj, gates, state, state_slots, cu_seqlens, out, heads, vdim, 2 * heads * (dim + vdim),
+                          heads * (vdim + 1) * dp + heads)
+        for n, t, size in (("gate_bias", gate_bias, 2 * heads), ("gain", gain, heads * vdim)):
+            _check(t, "matrix_memory." + n, torch.float32, 1)
+            _need(t.shape[0] == size, f"matrix_memory.{n}: {size} numbers")
+        tokens, requests, code, ld = proj.shape[0], state_slots.shape[0], DTYPE_CODE[proj.dtype], proj.shape[1]
+        scale = dim ** -0.5
+        if longest == 1 and tokens == requests:
+            self._call("llm_matrix_memory_step", _ptr(proj), ld, _ptr(gates), _ptr(gate_bias), float(cap), _ptr(gain), float(eps), float(tiny),
+                       _ptr(state), state.shape[1], _ptr(state_slots), _ptr(cu_seqlens), _ptr(out), code, requests, heads, dim, vdim, scale,
+                       1 if write else 0, self._stream())
+            return out
+        g4 = self._scratch("state.gates", 4 * tokens * heads, proj.device)
+        o = self._scratch("state.o", tokens * heads * (vdim + 1), proj.device)
+        self._call("llm_memory_gates", _ptr(gates), _ptr(gate_bias), float(cap), _ptr(state), state.shape[1], heads * (vdim + 1) * dp,
+                   _ptr(state_slots), _ptr(cu_seqlens), _ptr(g4), requests, heads, 1 if write else 0, self._stream())
+        walks, n_walks = self._state_walks(plan, requests)
+        self._call("llm_state_walk", 0, _ptr(proj), ld, _ptr(g4), None, None, _ptr(state), state.shape[1], _ptr(state_slots), _ptr(cu_seqlens),
+                   _ptr(walks), n_walks, _ptr(o), code, heads, heads, dim, vdim, scale, 1 if write else 0, self._stream())
+        self._call("llm_state_finish", 0, _ptr(o), _ptr(g4), _ptr(proj), ld, 2 * heads * dim + heads * vdim, _ptr(gain), _ptr(out), code, tokens,
+                   heads, vdim, float(eps), float(tiny), self._stream())
+        return out
+
+    def gated_delta(self, proj, gates, conv, rate, dt_bias, gain, eps: float, tiny: float, state, state_slots, positions, token_request,
+                    cu_seqlens, out, heads, kv_heads, dim, vdim, longest: int, plan=None, write: bool = True):
+        """A gated delta rule behind short convolutions (csrc/matrix_state.cu): proj [T, 2 * kv_heads * dim + 2 * heads * vdim] holds q,
+        k, v and the output gate's input; gates float32 [T, 2 * heads] (the step sizes' products, then the decays'); conv float32
+        [channels, taps]; rate, dt_bias [heads]; gain [vdim]; state float32 [slots, record]: per head vdim columns of dim numbers
+        (padded to four), then `taps` rows of the projection's channels (position p in row p % taps).  The state as in `matrix_memory`."""
+        dp, channels = -(-dim // 4) * 4, 2 * kv_heads * dim + heads * vdim
+        _check(conv, "gated_delta.conv", torch.float32, 2)
+        taps = conv.shape[1]
+        self._check_state("gated_delta", proj, gates, state, state_slots, cu_seqlens, out, heads, vdim, channels + heads * vdim,
+                          heads * vdim * dp + taps * channels)
+        _need(conv.shape[0] == channels and heads % kv_heads == 0, "gated_delta.conv: one row per channel of q, k and v")
+        for n, t, size in (("rate", rate, heads), ("dt_bias", dt_bias, heads), ("gain", gain, vdim)):
+            _check(t, "gated_delta." + n, torch.float32, 1)
+            _need(t.shape[0] == size, f"gated_delta.{n}: {size} numbers")
+        tokens, requests, code, ld = proj.shape[0], state_slots.shape[0], DTYPE_CODE[proj.dtype], proj.shape[1]
+        for n, t in (("positions", positions), ("token_request", token_request)):
+            _check(t, "gated_delta." + n, torch.int32, 1)
+            _need(t.shape[0] == tokens, f"gated_delta.{n}: one per token")
+        scale = dim ** -0.5
+        if longest == 1 and tokens == requests:
+            self._call("llm_gated_delta_step", _ptr(proj), ld, _ptr(gates), _ptr(conv), taps, _ptr(rate), _ptr(dt_bias), _ptr(gain), float(eps),
+                       float(tiny), _ptr(state), state.shape[1], _ptr(state_slots), _ptr(positions), _ptr(cu_seqlens), _ptr(out), code,
+                       requests, heads, kv_heads, dim, vdim, scale, 1 if write else 0, self._stream())
+            return out
+        n = tokens * channels
+        c = self._scratch("state.conv", n, proj.device) if code == 0 else self._scratch_bf16("state.conv", n, proj.device)
+        unit, steps = self._scratch("state.unit", 2 * tokens * kv_heads, proj.device), self._scratch("state.steps", 2 * tokens * heads, proj.device)
+        o = self._scratch("state.o", tokens * heads * vdim, proj.device)
+        self._call("llm_delta_prepare", _ptr(proj), ld, _ptr(gates), _ptr(conv), taps, _ptr(rate), _ptr(dt_bias), _ptr(state), state.shape[1],
+                   _ptr(state_slots), _ptr(positions), _ptr(token_request), _ptr(cu_seqlens), _ptr(c), _ptr(unit), _ptr(steps), code, tokens,
+                   requests, heads, kv_heads, dim, vdim, float(tiny), scale, 1 if write else 0, self._stream())
+        walks, n_walks = self._state_walks(plan, requests)
+        self._call("llm_state_walk", 1, _ptr(c), channels, None, _ptr(unit), _ptr(steps), _ptr(state), state.shape[1], _ptr(state_slots),
+                   _ptr(cu_seqlens), _ptr(walks), n_walks, _ptr(o), code, heads, kv_heads, dim, vdim, scale, 1 if write else 0, self._stream())
+        self._call("llm_state_finish", 1, _ptr(o), None, _ptr(proj), ld, channels, _ptr(gain), _ptr(out), code, tokens, heads, vdim,
+                   float(eps), float(tiny), self._stream())
         return out
 
     def token_shift(self, x, mu, before, state_slots, token_request, cu_seqlens, out):

@@ -11,10 +11,12 @@ from .base import ParamSpec, Part, StepPlan, StepShape
 from .block import (Arrangement, BranchNormBlock, BranchNormMixerBlock, PostNormDepthBlock, PostNormDepthMixerBlock, PreNormBlock,
                     PreNormMixerBlock, SandwichBlock, SandwichMixerBlock, SandwichMixerSideBlock, SandwichSideBlock)
 from .embedding import Embedding, NormedEmbedding, OutputHead, SideTableEmbedding, TanhNormedEmbedding
+from .delta_rule import GatedDelta
 from .feed_forward import GLU, ClampedGLU, PolyNormMLP, RoutedGLU, SwiGLU
 from .gated_attention import GatedAttention
 from .latent_attention import LatentAttention
 from .lru import GatedLRU
+from .matrix_memory import MatrixMemory
 from .mixer import PagedAttention
 from .parallel import ParallelMixer
 from .retention import Retention
@@ -31,7 +33,7 @@ NORMS = {"rmsnorm": RMSNorm, "rmsnorm_scalar": ScalarGainRMSNorm, "rmsnorm_one_p
 POSITION_ENCODINGS = {"rope": RotaryEmbedding, "none": NoPosition}
 MIXERS = {"attention": PagedAttention, "talking_attention": TalkingAttention, "retention": Retention,
           "latent_attention": LatentAttention, "gated_attention": GatedAttention, "wkv": WKV, "gated_lru": GatedLRU,
-          "parallel": ParallelMixer}
+          "parallel": ParallelMixer, "matrix_memory": MatrixMemory, "gated_delta": GatedDelta}
 FEED_FORWARDS = {"swiglu": SwiGLU, "glu": GLU, "clamped_glu": ClampedGLU, "routed_glu": RoutedGLU, "poly_norm_mlp": PolyNormMLP}
 ARRANGEMENTS = {"prenorm": PreNormBlock, "prenorm_mixer": PreNormMixerBlock, "branchnorm": BranchNormBlock,
                 "branchnorm_mixer": BranchNormMixerBlock, "sandwich": SandwichBlock, "sandwich_mixer": SandwichMixerBlock,

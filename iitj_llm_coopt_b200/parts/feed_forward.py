@@ -137,6 +137,9 @@ class RoutedGLU(Part):
     `correction` = False: there is no stored correction and the choice is by s alone; `expert` = "silu" makes the
     experts plain silu-gated ones, silu(g) * u, instead of the clamped form; `groups` = (count, keep): the router outputs form
     `count` equal groups of neighbours and only those of the `keep` groups with the largest single score can be chosen;
+    `group_worth` = 2: a group is worth the sum of its two largest scores instead of the largest alone;
+    `weight_scale` multiplies the chosen scores; `shared` = inner width of one more expert that every token uses with weight one
+    (silu-gated; its result is added to the weighted sum);
     `renormalize` = tiny: the chosen scores are divided by (their sum + tiny); `weight_on` = "input" feeds expert e the row
     s[e] * x and sums the experts' outputs as they are, out = sum expert_e(s[e] * x) (the first product being linear in
     its row, the weight is applied to gate and up in that product's epilogue, or to the gathered rows).
@@ -180,7 +183,14 @@ class RoutedGLU(Part):
             raise ValueError(f"routed feed-forward: {self.top} of {outputs} router outputs from groups {self.groups}")
         if self.chosen_softmax and (self.renormalize is not None or self.groups):
             raise ValueError("routed feed-forward: router = chosen_softmax takes neither groups nor a renormalisation")
+        self.group_worth, self.weight_scale = int(spec.option("group_worth", 1)), float(spec.option("weight_scale", 1.0))
+        if self.group_worth not in (1, 2) or (self.chosen_softmax and self.weight_scale != 1.0):
+            raise ValueError("routed feed-forward: group_worth is 1 or 2, weight_scale goes with scores of single outputs")
+        self.shared = int(spec.option("shared", 0))
+        if self.shared and (self.identity or not self.experts):
+            raise ValueError("routed feed-forward: a shared expert goes with experts that have tensors")
         self.router = self.correction = self.router_bias = self.expert_gate_up = self.expert_down = None
+        self.shared_gate_up = self.shared_down = None
         self.prepare_key = f"routed_glu.{self.top}"          # layers with as many choices a token share the step's plan
 
     def _by_expert(self, tokens: int) -> bool:
@@ -209,6 +219,10 @@ class RoutedGLU(Part):
             out["expert_gate_up"] = ParamSpec((e * 2 * ff, w), pieces=tuple(
                 (f"e{j}.{name}", ff) for j in range(e) for name in ("gate", "up")))
             out["expert_down"] = ParamSpec((e * w, ff), pieces=tuple((f"e{j}.down", w) for j in range(e)))
+        shared = int(spec.option("shared", 0))
+        if shared:
+            out["shared_gate_up"] = ParamSpec((2 * shared, w), pieces=(("gate", shared), ("up", shared)))
+            out["shared_down"] = ParamSpec((w, shared))
         return out
 
     def load(self, tensors: dict) -> None:
@@ -228,6 +242,8 @@ class RoutedGLU(Part):
             self.k.route_topk(scores, self.router_bias, chosen, weights, chosen_softmax=True)
         else:
             more = {} if not self.groups and self.renormalize is None else {"groups": self.groups, "renormalize": self.renormalize}
+            if self.group_worth != 1 or self.weight_scale != 1.0:
+                more.update(worth=self.group_worth, scale=self.weight_scale)
             self.k.route_topk(scores, self.correction, chosen, weights, sigmoid=self.sigmoid, **more)
         out = ctx.buffer("ffn.out", (t, self.width), self.dtype)
         plan = y = None
@@ -268,5 +284,9 @@ class RoutedGLU(Part):
                 self.k.moe_linear(x, w1, act, plan, gather=True, glu=glu, limit=self.limit,
                                   slope=self.slope)
                 self.k.moe_linear(act, w2, y, plan)
-        return self.k.moe_combine(y, plan, chosen, None if self.on_input else weights, x, self.experts, out,
-                                  **({"defer": True} if self.experts and not self.identity else {}))
+        more = {"defer": True} if self.experts and not self.identity else {}
+        if self.shared:      # its product comes last: the parts it may leave stand until the next split product
+            act = ctx.buffer("ffn.shared.act", (t, self.shared), self.dtype)
+            self.k.linear(x, self.shared_gate_up, act, swiglu=True)
+            more["extra"] = self.k.linear(act, self.shared_down, ctx.buffer("ffn.shared.out", (t, self.width), self.dtype), defer=True)
+        return self.k.moe_combine(y, plan, chosen, None if self.on_input else weights, x, self.experts, out, **more)

@@ -2,7 +2,8 @@
 
 y = x * rsqrt(mean(x^2) + eps) * weight  (engine/model.py:85-89), statistics in float32.
 The reference's fused form `residual += x; x = norm(residual)` (engine/model.py:236, 249, 254)
-is the `delta` argument here.
+is the `delta` argument here.  An option `branch_factor` of an RMSNorm's spec multiplies the delta on its way into the residual,
+residual += branch_factor * delta; the delta may then also be a routed feed-forward whose weighted sum is still to be taken.
 """
 from __future__ import annotations
 
@@ -16,15 +17,22 @@ class RMSNorm(Part):
     def __init__(self, spec, kernels, dtype):
         self.spec, self.k, self.dtype = spec, kernels, dtype
         self.width, self.eps = spec.width, spec.eps
+        self.factor = dict(spec.options).get("branch_factor")
+        self.takes_routed_sums = self.factor is not None
         self.weight = None
 
     @classmethod
     def parameters(cls, spec) -> dict:
         return {"weight": ParamSpec((spec.width,), kind="vector")}
 
+    def load(self, tensors: dict) -> None:
+        self.weight = tensors["weight"] if self.factor is None else tensors["weight"].float().contiguous()
+
     def forward(self, ctx, residual, delta=None, rows=None):
         n = rows.shape[0] if rows is not None else residual.shape[0]
         out = ctx.buffer(f"norm.{self.part_name}.out" if rows is None else f"norm.{self.part_name}.rows", (n, self.width), self.dtype)
+        if self.factor is not None and delta is not None:
+            return self.k.add_branch_rmsnorm(residual, delta, float(self.factor), self.weight, self.eps, out, rows=rows)
         return self.k.add_rmsnorm(residual, delta, self.weight, self.eps, out, rows=rows)
 
 

@@ -313,24 +313,24 @@ def ref_attention_flat(q, q_stride_heads, cache, block_table, token_request, pos
     return out.view(T, heads * value_dim)
 
 
-def ref_route_topk(scores, correction, top, sigmoid=False, chosen_softmax=False, groups=None, renormalize=None):
+def ref_route_topk(scores, correction, top, sigmoid=False, chosen_softmax=False, groups=None, renormalize=None, worth=1, scale=1.0):
     if chosen_softmax:             # the outputs (plus their bias) compared as they are; softmax over the chosen alone
         z = scores.float() + (correction.float() if correction is not None else 0.0)
         val, chosen = torch.topk(z, top, dim=-1)
         return chosen.to(torch.int32), torch.softmax(val, dim=-1)
     s = torch.sigmoid(scores.float()) if sigmoid else torch.softmax(scores.float(), dim=-1)
     c = s + correction.float() if correction is not None else s
-    if groups:                     # only entries of the groups with the largest single entry can be chosen
+    if groups:                     # only entries of the groups with the largest entry (sum of the `worth` largest) can be chosen
         count, keep = groups
         parts = c.view(c.shape[0], count, -1)
-        best = torch.topk(parts.amax(-1), keep, dim=-1).indices
+        best = torch.topk(torch.topk(parts, min(worth, parts.shape[-1]), dim=-1).values.sum(-1), keep, dim=-1).indices
         shut = torch.ones(c.shape[0], count, dtype=torch.bool, device=c.device).scatter_(1, best, False)
         c = parts.masked_fill(shut.unsqueeze(-1), float("-inf")).reshape(c.shape)
     chosen = torch.topk(c, top, dim=-1).indices
     w = torch.gather(s, 1, chosen)
     if renormalize is not None:
         w = w / (w.sum(-1, keepdim=True) + renormalize)
-    return chosen.to(torch.int32), w
+    return chosen.to(torch.int32), w * scale
 
 
 # ---- the Bidinex family's kernels ------------------------------------------------------------------------------
@@ -481,6 +481,84 @@ def ref_wkv_scan(rkvg, decay, u, gain, eps, state, state_slots, cu_seqlens, head
     return o.reshape(T, n) * gain.float() * g, new
 
 
+# ---- matrix states with a record per request ---------------------------------------------------------------------
+
+def _record(state_row, heads, dim, vdim, columns):
+    """(view [heads, columns, dim] of the states' columns (a column's numbers padded to a multiple of four), what follows them)"""
+    pad = -(-dim // 4) * 4
+    n = heads * columns * pad
+    return state_row[:n].view(heads, columns, pad)[:, :, :dim], state_row[n:]
+
+
+def _unit_rms(o, eps):
+    return o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+
+
+def ref_matrix_memory(proj, gates, gate_bias, cap, gain, eps, tiny, state, state_slots, cu_seqlens, heads, dim, vdim, write=True):
+    """[T, heads * vdim] float32; `state` [slots, record] is read and, with `write`, left at each request's last token."""
+    T, H = proj.shape[0], heads
+    x, dev = proj.float(), proj.device
+    q = x[:, :H * dim].view(T, H, dim) * dim ** -0.5
+    k = x[:, H * dim:2 * H * dim].view(T, H, dim)
+    v = x[:, 2 * H * dim:2 * H * dim + H * vdim].view(T, H, vdim)
+    z = x[:, 2 * H * dim + H * vdim:2 * H * dim + 2 * H * vdim]
+    pre = cap * torch.tanh((gates.float() + gate_bias.float()) / cap)
+    gi, gf = pre[:, :H], torch.nn.functional.logsigmoid(pre[:, H:])
+    o = torch.zeros(T, H, vdim, dtype=torch.float32, device=dev)
+    cu = [int(c) for c in cu_seqlens]
+    for b in range(len(cu) - 1):
+        if cu[b + 1] <= cu[b]:
+            continue
+        cols, rest = _record(state[int(state_slots[b])], H, dim, vdim, vdim + 1)
+        S, n, m = cols[:, :vdim].clone(), cols[:, vdim].clone(), rest[:H].clone()
+        for t in range(cu[b], cu[b + 1]):
+            new = torch.maximum(gf[t] + m, gi[t])
+            keep, add = torch.exp(gf[t] + m - new).view(H, 1), torch.exp(gi[t] - new).view(H, 1)
+            m = new
+            S = keep.unsqueeze(2) * S + (add * v[t]).unsqueeze(2) * k[t].unsqueeze(1)
+            n = keep * n + add * k[t]
+            den = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + tiny
+            o[t] = torch.einsum("hvd,hd->hv", S, q[t]) / den.view(H, 1)
+        if write:
+            cols[:, :vdim], cols[:, vdim], rest[:H] = S, n, m
+    return _unit_rms(o, eps).reshape(T, H * vdim) * gain.float() * torch.sigmoid(z)
+
+
+def ref_gated_delta(proj, gates, conv, rate, dt_bias, gain, eps, tiny, state, state_slots, positions, cu_seqlens, heads, kv_heads, dim,
+                    vdim, write=True):
+    """[T, heads * vdim] float32; `state` as above, the convolution's rows behind the states' columns (position p in row p % taps)."""
+    T, H, G, taps = proj.shape[0], heads, kv_heads, conv.shape[1]
+    x, dev, C = proj.float(), proj.device, 2 * G * dim + H * vdim
+    z = x[:, C:C + H * vdim].view(T, H, vdim)
+    beta = torch.sigmoid(gates[:, :H].float())
+    g = torch.exp(-rate.float() * torch.nn.functional.softplus(gates[:, H:].float() + dt_bias.float()))
+    o = torch.zeros(T, H, vdim, dtype=torch.float32, device=dev)
+    cu = [int(c) for c in cu_seqlens]
+    for b in range(len(cu) - 1):
+        if cu[b + 1] <= cu[b]:
+            continue
+        cols, rest = _record(state[int(state_slots[b])], H, dim, vdim, vdim)
+        ring, p0, S = rest[:taps * C].view(taps, C), int(positions[cu[b]]), cols.clone()
+        rows = {p: ring[p % taps].clone() for p in range(p0 - taps + 1, p0)}
+        for t in range(cu[b], cu[b + 1]):
+            p = p0 + t - cu[b]
+            rows[p] = x[t, :C]
+            c = torch.nn.functional.silu(sum(conv[:, j].float() * rows[p - taps + 1 + j] for j in range(taps)))
+            q, k, v = c[:G * dim].view(G, dim), c[G * dim:2 * G * dim].view(G, dim), c[2 * G * dim:].view(H, vdim)
+            q = (q * torch.rsqrt((q * q).sum(-1, keepdim=True) + tiny) * dim ** -0.5).repeat_interleave(H // G, dim=0)
+            k = (k * torch.rsqrt((k * k).sum(-1, keepdim=True) + tiny)).repeat_interleave(H // G, dim=0)
+            S = g[t].view(H, 1, 1) * S
+            u = beta[t].view(H, 1) * (v - torch.einsum("hvd,hd->hv", S, k))
+            S = S + u.unsqueeze(2) * k.unsqueeze(1)
+            o[t] = torch.einsum("hvd,hd->hv", S, q)
+        if write:
+            cols.copy_(S)
+            last = p0 + cu[b + 1] - cu[b]
+            for p in range(max(last - taps, p0), last):
+                ring[p % taps] = rows[p]
+    return (_unit_rms(o, eps) * gain.float() * torch.nn.functional.silu(z)).reshape(T, H * vdim)
+
+
 _M64 = np.uint64(0xFFFFFFFFFFFFFFFF)
 
 
@@ -528,6 +606,20 @@ class TorchKernels:
         if rows is None and delta is not None:
             residual.copy_(v)
         out.copy_(y)
+        return out
+
+    def add_branch_rmsnorm(self, residual, delta, factor, weight, eps, out, rows=None):
+        return self.add_rmsnorm(residual, factor * delta.float(), weight, eps, out, rows)
+
+    def matrix_memory(self, proj, gates, gate_bias, cap, gain, eps, tiny, state, state_slots, cu_seqlens, out, heads, dim, vdim,
+                      longest=0, plan=None, write=True):
+        out.copy_(ref_matrix_memory(proj, gates, gate_bias, cap, gain, eps, tiny, state, state_slots, cu_seqlens, heads, dim, vdim, write))
+        return out
+
+    def gated_delta(self, proj, gates, conv, rate, dt_bias, gain, eps, tiny, state, state_slots, positions, token_request, cu_seqlens,
+                    out, heads, kv_heads, dim, vdim, longest=0, plan=None, write=True):
+        out.copy_(ref_gated_delta(proj, gates, conv, rate, dt_bias, gain, eps, tiny, state, state_slots, positions, cu_seqlens, heads,
+                                  kv_heads, dim, vdim, write))
         return out
 
     def add_dynamic_tanh(self, residual, delta, factor, norm, out, rows=None, store=True):
@@ -726,8 +818,9 @@ class TorchKernels:
                           state, state_slots, cu_seqlens, write))
         return out
 
-    def route_topk(self, scores, correction, chosen, weights, sigmoid=False, chosen_softmax=False, groups=None, renormalize=None):
-        c, w = ref_route_topk(scores, correction, chosen.shape[1], sigmoid, chosen_softmax, groups, renormalize)
+    def route_topk(self, scores, correction, chosen, weights, sigmoid=False, chosen_softmax=False, groups=None, renormalize=None,
+                   worth=1, scale=1.0):
+        c, w = ref_route_topk(scores, correction, chosen.shape[1], sigmoid, chosen_softmax, groups, renormalize, worth, scale)
         chosen.copy_(c)
         weights.copy_(w)
 
@@ -785,7 +878,7 @@ class TorchKernels:
             out[r0:r0 + n] = y
         return out
 
-    def moe_combine(self, y, plan, chosen, weights, x, experts, out, defer=False):     # always summed at once
+    def moe_combine(self, y, plan, chosen, weights, x, experts, out, defer=False, extra=None):     # always summed at once
         T, top = chosen.shape
         acc = torch.zeros(T, x.shape[1], dtype=torch.float32, device=x.device)
         for t in range(T):
@@ -793,7 +886,7 @@ class TorchKernels:
                 e = int(chosen[t, j])
                 row = x[t].float() if e >= experts else y[int(plan["place"][t * top + j])].float()
                 acc[t] += (float(weights[t, j]) if weights is not None else 1.0) * row
-        out.copy_(acc)
+        out.copy_(acc if extra is None else acc + extra.float())
         return out
 
     def token_shift(self, x, mu, before, state_slots, token_request, cu_seqlens, out):
