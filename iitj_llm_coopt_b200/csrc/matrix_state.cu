@@ -348,8 +348,8 @@ struct WalkArgs {
     const int* state_slots;
     const int* cu_seqlens;
     const int* walks;                  // requests to walk (null: all)
-    float* o;                          // [tokens, heads, columns]
-    int heads, kv_heads, dim, vdim, write, ds;
+    float* o;                          // [tokens, heads, o_ld]
+    int heads, kv_heads, dim, vdim, o_ld, write, ds;
     float q_scale;
 };
 
@@ -443,7 +443,7 @@ state_walk_kernel(WalkArgs a) {
                     o[j] += __shfl_xor_sync(0xffffffffu, o[j], x);
                     if (KIND == kDelta) pk[j] += __shfl_xor_sync(0xffffffffu, pk[j], x);
                 }
-            float* o_at = a.o + ((size_t)(t0 + tt) * a.heads + h) * columns + c0;
+            float* o_at = a.o + ((size_t)(t0 + tt) * a.heads + h) * a.o_ld + c0;
 #pragma unroll
             for (int j = 0; j < COLS; ++j) {
                 if (KIND == kDelta) {
@@ -471,7 +471,7 @@ state_walk_kernel(WalkArgs a) {
 // out = (head of o / root mean square) * gain * gate; memory: o is divided by its normaliser first.  A warp per (token, head).
 template <typename T, int KIND>
 __global__ void __launch_bounds__(256)
-state_finish_kernel(const float* __restrict__ o, const float4* __restrict__ gates, const T* __restrict__ proj, int ld, int z_col,
+state_finish_kernel(const float* __restrict__ o, int o_ld, const float4* __restrict__ gates, const T* __restrict__ proj, int ld, int z_col,
                     const float* __restrict__ gain, T* __restrict__ out, int heads, int vdim, float eps, float tiny, long long rows) {
     pdl_trigger();
     pdl_wait();
@@ -479,8 +479,7 @@ state_finish_kernel(const float* __restrict__ o, const float4* __restrict__ gate
     if (row >= rows) return;
     const int lane = threadIdx.x & 31, h = (int)(row % heads);
     const long long t = row / heads;
-    const int columns = KIND == kMemory ? vdim + 1 : vdim;
-    const float* x = o + row * columns;
+    const float* x = o + row * o_ld;
     float den = 1.f;
     if (KIND == kMemory) den = 1.0f / (fmaxf(fabsf(x[vdim]), expf(-gates[row].z)) + tiny);
     float ss = 0.f;
@@ -621,22 +620,22 @@ LLM_API int llm_delta_prepare(const void* proj, int ld, const float* gates, cons
 // kind 0: matrix memory (gates), kind 1: gated delta rule (unit, steps).  walks: null (all of `n_walks` requests) or their indices.
 LLM_API int llm_state_walk(int kind, const void* qkv, int ld, const void* gates, const void* unit, const void* steps, float* state,
                            long long slot_stride, const int* state_slots, const int* cu_seqlens, const int* walks, int n_walks, float* o,
-                           int dtype, int heads, int kv_heads, int dim, int vdim, float q_scale, int write, cudaStream_t stream) {
+                           int o_ld, int dtype, int heads, int kv_heads, int dim, int vdim, float q_scale, int write, cudaStream_t stream) {
     if (n_walks == 0) return 0;
     if (dim > 1024 || dim <= 0 || vdim <= 0) LLM_FAIL(-1, "state_walk: head sizes %d / %d (1 to 1024 rows)", dim, vdim);
     WalkArgs a{qkv, ld, (const float4*)gates, (const float2*)unit, (const float2*)steps, state, slot_stride, state_slots, cu_seqlens, walks, o,
-               heads, kv_heads, dim, vdim, write, 8, q_scale};
+               heads, kv_heads, dim, vdim, o_ld, write, 8, q_scale};
     return kind == kMemory ? run_walk<kMemory>(a, dtype, n_walks, stream) : run_walk<kDelta>(a, dtype, n_walks, stream);
 }
 
-LLM_API int llm_state_finish(int kind, const float* o, const void* gates, const void* proj, int ld, int z_col, const float* gain, void* out,
+LLM_API int llm_state_finish(int kind, const float* o, int o_ld, const void* gates, const void* proj, int ld, int z_col, const float* gain, void* out,
                              int dtype, int tokens, int heads, int vdim, float eps, float tiny, cudaStream_t stream) {
     if (tokens == 0) return 0;
     const long long rows = (long long)tokens * heads;
     return llm_dispatch_dtype(dtype, [&](auto tag) {
         using T = decltype(tag);
         auto go = [&](auto kern) {
-            llm_launch(kern, (unsigned)((rows + 7) / 8), 256, 0, stream, o, (const float4*)gates, (const T*)proj, ld, z_col, gain, (T*)out, heads,
+            llm_launch(kern, (unsigned)((rows + 7) / 8), 256, 0, stream, o, o_ld, (const float4*)gates, (const T*)proj, ld, z_col, gain, (T*)out, heads,
                        vdim, eps, tiny, rows);
         };
         if (kind == kMemory) go(state_finish_kernel<T, kMemory>);

@@ -809,6 +809,132 @@ def _kernels_alone_bidinex(cfg, beside, tokens, batch, context, hbm_gbs, flush):
     return out
 
 
+def _kernels_alone_kobolix(cfg, beside, tokens, batch, context, hbm_gbs, flush):
+    """The kernels and kernel options that Kobolix brought, alone at the shapes of a `tokens`-token prompt and of a decode step of
+    `batch` requests, each beside the like kernel as Mamusun, Rodapel, Bidinex or Llama runs it: microseconds, the bytes that must move
+    and the fraction of the copy bandwidth that is, and for the recurrences the TFLOP/s of the token-by-token form's arithmetic."""
+    import torch
+
+    from . import kernels as _k
+    from .parts.base import StepShape
+    from .parts.delta_rule import record as delta_record
+    from .parts.matrix_memory import record as memory_record
+    from .parts.state_plan import plan_state_chunks
+    K = _k.load()
+    dev, bf = "cuda", torch.bfloat16
+    mem = next(l["mixer"] for l in cfg["layers"] if l["type"] == "mlstm")
+    par = next(l["mixer"] for l in cfg["layers"] if l["type"] == "parallel")
+    moe = next(l["mlp"] for l in cfg["layers"] if l["mlp"]["kind"] == "moe")
+    lru = next(l["mixer"]["right"] for l in beside["layers"] if l["type"] == "parallel")
+    width, left, right, page, out = cfg["width"], par["left"], par["right"], 16, []
+
+    def i32(x):
+        return torch.tensor(x, dtype=torch.int32, device=dev)
+
+    def rand(*shape, s=1.0):
+        return (torch.randn(*shape, device=dev) * s).to(bf)
+
+    def record(name, fn, nbytes=None, flops=None, like=None, reps=10):
+        us = 1e3 * _timed(fn, reps, 3, flush)
+        r = {"kernel": name, "us": round(us, 2)}
+        if nbytes is not None:
+            r.update(mbytes=round(nbytes / 1e6, 2), frac_of_copy_bandwidth=round(nbytes / (us * 1e-6) / (hbm_gbs * 1e9), 3))
+        if flops is not None:
+            r.update(tflops=round(flops / (us * 1e-6) / 1e12, 2))
+        if like:
+            r["like"] = like
+        out.append(r)
+
+    for label, T, B, per in (("prefill", tokens, 1, tokens), ("decode", batch, batch, 1)):
+        ctx_len = per if label == "prefill" else context
+        treq = i32([b for b in range(B) for _ in range(per)])
+        pos_host = [ctx_len - per + i for _ in range(B) for i in range(per)]
+        pos, cu, slots = i32(pos_host), i32([per * b for b in range(B + 1)]), i32(list(range(B)))
+        plan = plan_state_chunks(K, StepShape([per] * B, [ctx_len] * B, T, label == "decode", False, dev))
+        if plan is not None:
+            plan.bind({k: i32(v) for k, v in plan.arrays.items()})
+        # --- matrix memory
+        H, D, V = mem["heads"], mem["dim"], mem["vdim"]
+        proj, gates = rand(T, 2 * H * (D + V)), torch.randn(T, 2 * H, device=dev)
+        bias, gain = torch.zeros(2 * H, device=dev), torch.ones(H * V, device=dev)
+        bias[H:] = 4.0
+        state, o = torch.zeros(B + 1, memory_record(H, D, V), device=dev), torch.empty(T, H * V, device=dev, dtype=bf)
+        record(f"matrix_memory ({label})",
+               lambda: K.matrix_memory(proj, gates, bias, mem["gate_cap"], gain, 1e-6, 1e-6, state, slots, cu, o, H, D, V, longest=per, plan=plan),
+               T * H * (2 * D + 3 * V) * 2 + 2 * B * H * (V + 1) * D * 4, 5 * T * H * D * V, like=f"wkv_scan ({label})", reps=5)
+        # --- gated delta rule with its convolutions
+        RH, RG, RD, RV, taps = (right[k] for k in ("heads", "kv_heads", "dim", "vdim", "conv"))
+        C = 2 * RG * RD + RH * RV
+        rproj, rgates = rand(T, C + RH * RV), torch.randn(T, 2 * RH, device=dev)
+        conv, rate, dt, rgain = torch.randn(C, taps, device=dev) * 0.5, torch.ones(RH, device=dev), torch.zeros(RH, device=dev), torch.ones(RV, device=dev)
+        rstate, ro = torch.zeros(B + 1, delta_record(RH, RG, RD, RV, taps), device=dev), torch.empty(T, RH * RV, device=dev, dtype=bf)
+        record(f"gated_delta with its convolutions ({label})",
+               lambda: K.gated_delta(rproj, rgates, conv, rate, dt, rgain, 1e-6, 1e-6, rstate, slots, pos, treq, cu, ro, RH, RG, RD, RV, longest=per,
+                                     plan=plan), T * (C + 2 * RH * RV) * 2 + B * (2 * RH * RV * RD + taps * C) * 4, 7 * T * RH * RD * RV,
+               like=f"wkv_scan ({label})", reps=5)
+        # --- the recurrences of the other families: a matrix state per head, the linear recurrence that stands in Mamusun's place
+        rn = 64 * (width // 64)
+        rkvg, decay, wst = rand(4 * T, rn), torch.rand(T, rn, device=dev), torch.zeros(B, rn // 64, 64, 64, device=dev)
+        wo = torch.empty(T, rn, device=dev, dtype=bf)
+        record(f"wkv_scan ({label})", lambda: K.wkv_scan(rkvg, decay, torch.zeros(rn // 64, 64, device=dev), torch.ones(rn, device=dev), 1e-6, wst, slots,
+                                                         cu, wo, rn // 64, 64), T * rn * (8 + 4 + 2) + B * rn * 64 * 8, 7 * T * rn * 64, reps=5)
+        inner, blocks, ltaps = lru["width"], lru["blocks"], lru["conv"]
+        lproj, lst, vec = rand(T, 2 * inner), torch.zeros(B, ltaps, inner, device=dev), torch.zeros(inner, device=dev)
+        ra = rand(blocks, inner // blocks, inner // blocks, s=0.05)
+        lo = torch.empty(T, inner, device=dev, dtype=bf)
+        record(f"lru with its convolution and gates ({label})",
+               lambda: K.lru(lproj, 0, inner, inner, vec, vec, torch.randn(inner, ltaps, device=dev), vec, ra, ra, vec, vec, vec, 8.0, lst, slots, treq, cu,
+                             lo, longest=per), T * inner * 6 + 4 * ra.numel() + B * ltaps * inner * 8, reps=5)
+        # --- the attention's rotation of neighbours without norms
+        AH, AG, AD, AV = (left[k] for k in ("heads", "kv_heads", "dim", "vdim"))
+        rot = left["rot"]["dims"]
+        pages = -(-ctx_len // page)
+        slot = i32([(b * pages + p // page) * page + p % page for b, p in zip(treq.tolist(), pos_host)])
+        cache, qkv = torch.zeros(B * pages + 1, AG * page * (AD + AV), device=dev, dtype=bf), rand(T, AH * AD + AG * (AD + AV))
+        ang = pos.float().unsqueeze(1) * (1.0 / 5e5 ** (torch.arange(rot // 2, device=dev).float() / (rot // 2)))
+        tabs = (ang.cos().contiguous(), ang.sin().contiguous())
+        moved = T * (AH * AD + AG * (AD + AV)) * 2 * 2
+        for norm in ("none", "head"):
+            record(f"qk_prepare, neighbours rotate{', then unit head norms' if norm == 'head' else ''} ({label})",
+                   lambda: K.qk_prepare(qkv, AH, AG, AD, AV, 1e-6, cache_layer=cache, slots=slot, norm=norm, norm_first=False, tables=tabs,
+                                        rotary_dim=rot, interleaved=True), moved,
+                   like=f"qk_prepare, neighbours rotate, then unit head norms ({label})" if norm == "none" else None)
+        # --- the branch norm with every form of the branch
+        res, branch, nw = torch.randn(T, width, device=dev), rand(T, width), torch.ones(width, device=dev)
+        xo = torch.empty(T, width, device=dev, dtype=bf)
+        record(f"add_branch_rmsnorm ({label})", lambda: K.add_branch_rmsnorm(res, branch, 0.5, nw, 1e-6, xo), T * width * 12,
+               like=f"add_rmsnorm ({label})")
+        record(f"add_rmsnorm ({label})", lambda: K.add_rmsnorm(res, branch, nw, 1e-6, xo), T * width * 12)
+        f32 = torch.randn(T, width, device=dev)
+        record(f"add_branch_rmsnorm, float32 rows ({label})", lambda: K.add_branch_rmsnorm(res, f32, 0.5, nw, 1e-6, xo), T * width * 14,
+               like=f"add_rmsnorm ({label})")
+        if label == "decode":
+            sums = _k.PartialSums(K, torch.randn(4, T, width, device=dev), xo)
+            record(f"add_branch_rmsnorm, four k-split parts ({label})", lambda: K.add_branch_rmsnorm(res, sums, 0.5, nw, 1e-6, xo), T * width * 26,
+                   like=f"add_rmsnorm, four k-split parts ({label})")
+            record(f"add_rmsnorm, four k-split parts ({label})", lambda: K.add_rmsnorm(res, sums, nw, 1e-6, xo), T * width * 26)
+        # --- routing and the routed branch with a shared expert's row
+        r = moe["router"]
+        E, top = r["experts"], r["top"]
+        scores = torch.randn(T, E, device=dev)
+        chosen, wts = torch.empty(T, top, dtype=torch.int32, device=dev), torch.empty(T, top, device=dev)
+        grp = (r["groups"]["count"], r["groups"]["keep"])
+        record(f"route_topk, sigmoid, groups by their two best ({label})",
+               lambda: K.route_topk(scores, None, chosen, wts, sigmoid=True, groups=grp, worth=2, scale=r["scale"]),
+               like=f"route_topk, softmax, best groups ({label})")
+        record(f"route_topk, softmax, best groups ({label})", lambda: K.route_topk(scores, None, chosen, wts, groups=grp, renormalize=1e-20))
+        rows = T * top
+        mp = K.moe_plan(chosen, E, i32([0] * rows), i32([0] * rows), torch.zeros(K.moe_tile_bound(rows, E) + 1, 4, dtype=torch.int32, device=dev))
+        y, shared = rand(rows, width), rand(T, width)
+        routed = K.moe_combine(y, mp, chosen, wts, branch, E, xo, defer=True, extra=shared)
+        plain = K.moe_combine(y, mp, chosen, wts, branch, E, xo, defer=True)
+        one = torch.ones(1, device=dev)
+        record(f"add_branch_rmsnorm, routed rows and a shared row ({label})", lambda: K.add_branch_rmsnorm(res, routed, 0.5, nw, 1e-6, xo),
+               ((rows + T) * 2 + T * 10) * width, like=f"add_dynamic_tanh, routed rows ({label})")
+        record(f"add_dynamic_tanh, routed rows ({label})", lambda: K.add_dynamic_tanh(res, plain, 0.5, (one, nw, nw), xo), (rows * 2 + T * 10) * width)
+    return out
+
+
 def run(family, shape, steps, warmup, batch, context, prefill_tokens, peaks_and_source) -> dict:
     import torch
 
@@ -826,14 +952,15 @@ def run(family, shape, steps, warmup, batch, context, prefill_tokens, peaks_and_
     rows = [_model_runs(f"{family}-{shape}", lif, lif["vocab"], batch, context, steps, warmup, prefill_tokens, flush)]
     beside = None
     # the closest family stands beside it too: windowed attention, a recurrence, routed experts; or latent attention and silu experts
-    close = {"fomerax": "rodapel", "mamusun": "rodapel", "bidinex": "fomerax"}.get(family)
+    close = {"fomerax": "rodapel", "mamusun": "rodapel", "bidinex": "fomerax", "kobolix": "mamusun"}.get(family)
     if close:
         _, beside = SHAPES[f"{close}-{shape}"]
         rows.append(_model_runs(f"{close}-{shape}", beside, beside["vocab"], batch, context, steps, warmup, prefill_tokens, flush))
     rows.append(_model_runs(f"{llama_name} cut to {depth} layers", llama, llama["vocab_size"], batch, context, steps, warmup,
                             prefill_tokens, flush))
     alone = {"lifusun": _kernels_alone_lifusun, "rodapel": _kernels_alone_rodapel, "fomerax": _kernels_alone_fomerax,
-             "mamusun": _kernels_alone_mamusun, "bidinex": _kernels_alone_bidinex}[family](
+             "mamusun": _kernels_alone_mamusun, "bidinex": _kernels_alone_bidinex,
+             "kobolix": _kernels_alone_kobolix}[family](
         lif, beside if beside is not None else llama, prefill_tokens, batch, context, peaks["hbm_gbs"], flush)
     return {"family": family, "shape": shape, "dtype": "bf16", "data": "synthetic (random weights, random tokens)",
             "models": rows, "kernels_alone": alone, "copy_bandwidth_gbs": peaks["hbm_gbs"], "peaks": f"of {source}",

@@ -168,8 +168,17 @@ _SIGNATURES = {
                           _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
                           _c_int, _c_int, _c_float, _c_float, _c_int, _c_void_p],
     "llm_state_walk": [_c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, ctypes.c_longlong, _c_void_p, _c_void_p,
-                       _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p],
-    "llm_state_finish": [_c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
+                       _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p],
+    "llm_state_chunk_tokens": [],
+    "llm_memory_chunk_supported": [_c_int, _c_int],
+    "llm_delta_chunk_supported": [_c_int, _c_int],
+    "llm_delta_chunk_tri_numbers": [],
+    "llm_delta_chunk_factor_numbers": [],
+    "llm_memory_chunks": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
+                          _c_void_p, ctypes.c_longlong, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p],
+    "llm_delta_chunks": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p,
+                         ctypes.c_longlong, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+    "llm_state_finish": [_c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
                          _c_float, _c_float, _c_void_p],
     "llm_token_shift": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
                         _c_void_p],
@@ -1464,9 +1473,16 @@ class Kernels:
             _check(t, f"{name}.{n}", torch.int32, 1)
         _need(cu_seqlens.shape[0] == state_slots.shape[0] + 1, name + ".cu_seqlens: requests + 1 entries")
 
-    def _state_walks(self, plan, requests):
-        """(device list of the requests that are walked token by token, their count): all without a plan"""
-        return (None, requests) if plan is None else (plan.device_arrays["walks"], plan.counts[0])
+    STATE_CHUNK = 64             # tokens of a chunk (csrc/matrix_state_mma.cu)
+    # tokens from which a request's portion is cut into chunks instead of walked (IITJ_STATE_CHUNK_FROM; 0: never)
+    state_chunk_from = int(os.environ.get("IITJ_STATE_CHUNK_FROM", "64")) or 1 << 30
+
+    def _state_parts(self, plan, requests, supported):
+        """(device list of the requests that are walked token by token, their count, the plan where long portions go by chunks): all
+        are walked without a plan, or where the chunked kernels do not take the sizes or the type."""
+        if plan is None or not plan.counts[1] or not supported:
+            return None, requests, None
+        return plan.device_arrays["walks"], plan.counts[0], plan
 
     def matrix_memory(self, proj, gates, gate_bias, cap: float, gain, eps: float, tiny: float, state, state_slots, cu_seqlens, out, heads,
                       dim, vdim, longest: int, plan=None, write: bool = True):
@@ -1489,13 +1505,24 @@ class Kernels:
                        1 if write else 0, self._stream())
             return out
         g4 = self._scratch("state.gates", 4 * tokens * heads, proj.device)
-        o = self._scratch("state.o", tokens * heads * (vdim + 1), proj.device)
+        o_ld = -(-(vdim + 1) // 4) * 4
+        o = self._scratch("state.o", tokens * heads * o_ld, proj.device)
         self._call("llm_memory_gates", _ptr(gates), _ptr(gate_bias), float(cap), _ptr(state), state.shape[1], heads * (vdim + 1) * dp,
                    _ptr(state_slots), _ptr(cu_seqlens), _ptr(g4), requests, heads, 1 if write else 0, self._stream())
-        walks, n_walks = self._state_walks(plan, requests)
-        self._call("llm_state_walk", 0, _ptr(proj), ld, _ptr(g4), None, None, _ptr(state), state.shape[1], _ptr(state_slots), _ptr(cu_seqlens),
-                   _ptr(walks), n_walks, _ptr(o), code, heads, heads, dim, vdim, scale, 1 if write else 0, self._stream())
-        self._call("llm_state_finish", 0, _ptr(o), _ptr(g4), _ptr(proj), ld, 2 * heads * dim + heads * vdim, _ptr(gain), _ptr(out), code, tokens,
+        walks, n_walks, chunked = self._state_parts(plan, requests, code == 1 and ld % 8 == 0 and self.lib.llm_memory_chunk_supported(dim, vdim))
+        if chunked is not None:
+            _, n_chunks, n_longs = chunked.counts
+            n = n_chunks * heads * (vdim + 1) * dim
+            own, decay = self._scratch("state.own", n, proj.device), self._scratch("state.decay", n_chunks * heads, proj.device)
+            hi, lo = self._scratch_bf16("state.hi", n, proj.device), self._scratch_bf16("state.lo", n, proj.device)
+            self._call("llm_memory_chunks", _ptr(proj), ld, _ptr(g4), _ptr(chunked.device_arrays["chunks"]), n_chunks,
+                       _ptr(chunked.device_arrays["longs"]), n_longs, _ptr(own), _ptr(hi), _ptr(lo), _ptr(decay), _ptr(state), state.shape[1],
+                       _ptr(state_slots), _ptr(o), o_ld, heads, dim, vdim, scale, 1 if write else 0, self._stream())
+            self.launches += 2
+        if n_walks:
+            self._call("llm_state_walk", 0, _ptr(proj), ld, _ptr(g4), None, None, _ptr(state), state.shape[1], _ptr(state_slots), _ptr(cu_seqlens),
+                       _ptr(walks), n_walks, _ptr(o), o_ld, code, heads, heads, dim, vdim, scale, 1 if write else 0, self._stream())
+        self._call("llm_state_finish", 0, _ptr(o), o_ld, _ptr(g4), _ptr(proj), ld, 2 * heads * dim + heads * vdim, _ptr(gain), _ptr(out), code, tokens,
                    heads, vdim, float(eps), float(tiny), self._stream())
         return out
 
@@ -1527,14 +1554,26 @@ class Kernels:
         n = tokens * channels
         c = self._scratch("state.conv", n, proj.device) if code == 0 else self._scratch_bf16("state.conv", n, proj.device)
         unit, steps = self._scratch("state.unit", 2 * tokens * kv_heads, proj.device), self._scratch("state.steps", 2 * tokens * heads, proj.device)
-        o = self._scratch("state.o", tokens * heads * vdim, proj.device)
+        o_ld = -(-vdim // 4) * 4
+        o = self._scratch("state.o", tokens * heads * o_ld, proj.device)
         self._call("llm_delta_prepare", _ptr(proj), ld, _ptr(gates), _ptr(conv), taps, _ptr(rate), _ptr(dt_bias), _ptr(state), state.shape[1],
                    _ptr(state_slots), _ptr(positions), _ptr(token_request), _ptr(cu_seqlens), _ptr(c), _ptr(unit), _ptr(steps), code, tokens,
                    requests, heads, kv_heads, dim, vdim, float(tiny), scale, 1 if write else 0, self._stream())
-        walks, n_walks = self._state_walks(plan, requests)
-        self._call("llm_state_walk", 1, _ptr(c), channels, None, _ptr(unit), _ptr(steps), _ptr(state), state.shape[1], _ptr(state_slots),
-                   _ptr(cu_seqlens), _ptr(walks), n_walks, _ptr(o), code, heads, kv_heads, dim, vdim, scale, 1 if write else 0, self._stream())
-        self._call("llm_state_finish", 1, _ptr(o), None, _ptr(proj), ld, channels, _ptr(gain), _ptr(out), code, tokens, heads, vdim,
+        self.launches += 1 if write else 0
+        walks, n_walks, chunked = self._state_parts(plan, requests, code == 1 and channels % 8 == 0 and self.lib.llm_delta_chunk_supported(dim, vdim))
+        if chunked is not None:
+            _, n_chunks, n_longs = chunked.counts
+            tri = self._scratch_bf16("state.tri", n_chunks * heads * self.lib.llm_delta_chunk_tri_numbers(), proj.device)
+            factors = self._scratch("state.factors", n_chunks * heads * self.lib.llm_delta_chunk_factor_numbers(), proj.device)
+            self._call("llm_delta_chunks", _ptr(c), channels, _ptr(unit), _ptr(steps), _ptr(chunked.device_arrays["chunks"]), n_chunks,
+                       _ptr(chunked.device_arrays["longs"]), n_longs, _ptr(tri), _ptr(factors), _ptr(state), state.shape[1], _ptr(state_slots),
+                       _ptr(o), o_ld, heads, kv_heads, dim, vdim, 1 if write else 0, self._stream())
+            self.launches += 1
+        if n_walks:
+            self._call("llm_state_walk", 1, _ptr(c), channels, None, _ptr(unit), _ptr(steps), _ptr(state), state.shape[1], _ptr(state_slots),
+                       _ptr(cu_seqlens), _ptr(walks), n_walks, _ptr(o), o_ld, code, heads, kv_heads, dim, vdim, scale, 1 if write else 0,
+                       self._stream())
+        self._call("llm_state_finish", 1, _ptr(o), o_ld, None, _ptr(proj), ld, channels, _ptr(gain), _ptr(out), code, tokens, heads, vdim,
                    float(eps), float(tiny), self._stream())
         return out
 

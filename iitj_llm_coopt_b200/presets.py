@@ -177,6 +177,35 @@ BIDINEX_3B = bidinex_shape(3072, 8192, 24, 128, 128256)
 BIDINEX_1B = bidinex_shape(2048, 8192, 32, 64, 128256)
 BIDINEX_TOY = bidinex_shape(512, 1408, 8, 64, 4096, layers=3, loop=(1, 2, 2), kv_rank=128, rot_dim=32, experts=4, groups=(2, 1))
 
+def kobolix_shape(width, inner, heads, kv_heads, head_dim, vocab, blocks, mem_heads, mem_dim, mem_vdim, delta_heads, delta_kv_heads,
+                  delta_dim, taps=4, experts=8, top=2, groups=(4, 2)) -> dict:
+    """A Kobolix config.json of `blocks` groups of four layers (matrix memory with a dense feed-forward, matrix memory with routed
+    experts, attention beside a delta rule with a dense one, matrix memory with routed experts) at the layer sizes of a Llama of the
+    same width: for runs with random weights beside the Mamusun and the Llama of that size.  A routed layer holds `experts` experts of
+    half the dense inner width and a shared one of a quarter."""
+    mem = {"heads": mem_heads, "dim": mem_dim, "vdim": mem_vdim, "gate_cap": 12.0}
+    par = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+                    "rot": {"dims": head_dim // 2, "base": 500000.0}},
+           "right": {"heads": delta_heads, "kv_heads": delta_kv_heads, "dim": delta_dim, "vdim": delta_dim, "conv": taps}}
+    dense = {"kind": "dense", "ff": inner}
+    routed = {"kind": "moe", "expert": {"ff": inner // 2}, "shared": {"ff": inner // 4},
+              "router": {"experts": experts, "top": top, "scale": 2.5, "groups": {"count": groups[0], "keep": groups[1]}}}
+    layers = []
+    for _ in range(blocks):
+        layers += [{"type": "mlstm", "mixer": dict(mem), "mlp": dict(dense)},
+                   {"type": "mlstm", "mixer": dict(mem), "mlp": copy.deepcopy(routed)},
+                   {"type": "parallel", "mixer": copy.deepcopy(par), "mlp": dict(dense)},
+                   {"type": "mlstm", "mixer": dict(mem), "mlp": copy.deepcopy(routed)}]
+    return {"architecture": "Kobolix", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+            "embedding": {"scale": 12.0}, "layers": layers}
+
+
+# Kobolix at the layer sizes of the Llama shapes above (8 layers each)
+KOBOLIX_8B = kobolix_shape(4096, 14336, 32, 8, 128, 128256, 2, 32, 64, 128, 32, 16, 128)
+KOBOLIX_3B = kobolix_shape(3072, 8192, 24, 8, 128, 128256, 2, 24, 64, 128, 24, 12, 128)
+KOBOLIX_1B = kobolix_shape(2048, 8192, 32, 8, 64, 128256, 2, 16, 64, 128, 32, 16, 64)
+KOBOLIX_TOY = kobolix_shape(512, 1408, 8, 2, 64, 4096, 1, 4, 64, 128, 8, 4, 64, experts=4, groups=(2, 1))
+
 # name -> (label used in reports, config.json dict)
 SHAPES = {
     "8b": ("llama-3.1-8b-shape-random", LLAMA_3_1_8B),
@@ -205,6 +234,10 @@ SHAPES = {
     "bidinex-3b": ("bidinex-3b-layers-random", BIDINEX_3B),
     "bidinex-1b": ("bidinex-1b-layers-random", BIDINEX_1B),
     "bidinex-toy": ("bidinex-toy-layers-random", BIDINEX_TOY),
+    "kobolix-8b": ("kobolix-8b-layers-random", KOBOLIX_8B),
+    "kobolix-3b": ("kobolix-3b-layers-random", KOBOLIX_3B),
+    "kobolix-1b": ("kobolix-1b-layers-random", KOBOLIX_1B),
+    "kobolix-toy": ("kobolix-toy-layers-random", KOBOLIX_TOY),
 }
 
 
