@@ -6,8 +6,8 @@
 //                   A block owns a head of a request, or a cluster of up to eight blocks shares it by columns and exchanges the head
 //                   norm's sums of squares.  A block asks for its first columns before it waits for the kernel ahead of it: a
 //                   state slot is written by this layer's kernels alone, in an earlier step.
-// llm_memory_gates: the gates of every token and the running maximum m along each request, a warp per request and head: m_t =
-//                   max(f_t + m_(t-1), i_t) is scanned with the pairs (sum of f, maximum), 32 tokens at a time.
+// llm_memory_gates: the gates of every token and the running maximum m along each request, a block per request and head: m_t =
+//                   max(f_t + m_(t-1), i_t) is scanned with the pairs (sum of f, maximum), 256 tokens at a time.
 // llm_delta_prepare: convolution, silu, unit lengths, decays and step sizes of every token; the convolution's rows it leaves behind
 //                   (llm_delta_rows) are written by a launch of their own, since other blocks of this one still read them.
 // llm_state_walk:   portions of prompts token by token: a block owns some columns of a head of a request in registers, a column's rows
@@ -18,6 +18,7 @@
 
 namespace {
 
+typedef __nv_bfloat16 bf16;
 constexpr int kStage = 16;             // tokens whose rows the walk stages at a time
 
 struct StepArgs {
@@ -235,15 +236,16 @@ state_step_kernel(StepArgs a) {
     }
 }
 
-// gates of the step's tokens [tokens, heads] as (f, i, m, m of the token before); a warp per request and head
-__global__ void __launch_bounds__(128)
+// gates of the step's tokens [tokens, heads] as (f, i, m, m of the token before); a block per request and head
+constexpr int kGateThreads = 256;
+__global__ void __launch_bounds__(kGateThreads)
 memory_gates_kernel(const float* __restrict__ gates, const float* __restrict__ bias, float cap, float* __restrict__ state,
                     long long slot_stride, long long m_offset, const int* __restrict__ state_slots, const int* __restrict__ cu_seqlens,
                     float4* __restrict__ out, int heads, int write) {
     pdl_trigger();
     pdl_wait();
-    const int b = blockIdx.x, h = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (h >= heads) return;
+    __shared__ float2 part[2][kGateThreads / 32];          // two buffers in turn: one barrier a round
+    const int b = blockIdx.x, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int lo = cu_seqlens[b], hi = cu_seqlens[b + 1];
     if (hi <= lo) return;
     float* m_at = state + (size_t)state_slots[b] * slot_stride + m_offset + h;
@@ -251,26 +253,34 @@ memory_gates_kernel(const float* __restrict__ gates, const float* __restrict__ b
     auto load = [&](int t) {
         return t < hi ? memory_gates(gates + (size_t)t * 2 * heads, bias, heads, h, cap) : make_float2(0.f, -INFINITY);
     };
-    float2 next = load(lo + lane);
-    for (int t0 = lo; t0 < hi; t0 += 32) {
+    float2 next = load(lo + threadIdx.x);
+    int turn = 0;
+    for (int t0 = lo; t0 < hi; t0 += kGateThreads, turn ^= 1) {
         const float2 g = next;
-        next = load(t0 + 32 + lane);
-        // (F, A): tokens up to this one turn m into max(F + m, A)
+        if (t0 + kGateThreads < hi) next = load(t0 + kGateThreads + threadIdx.x);
+        // (F, A): the warp's tokens up to this one turn m into max(F + m, A)
         float F = g.x, A = g.y;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const float Fb = __shfl_up_sync(0xffffffffu, F, o), Ab = __shfl_up_sync(0xffffffffu, A, o);
             if (lane >= o) { A = fmaxf(Ab + F, A); F += Fb; }
         }
-        const float m = fmaxf(F + m0, A);
+        if (lane == 31) part[turn][warp] = make_float2(F, A);
+        __syncthreads();
+        float start = m0;
+#pragma unroll
+        for (int w = 0; w < kGateThreads / 32; ++w) {
+            if (w == warp) start = m0;
+            m0 = fmaxf(part[turn][w].x + m0, part[turn][w].y);       // behind the last token nothing changes m
+        }
+        const float m = fmaxf(F + start, A);
         float before = __shfl_up_sync(0xffffffffu, m, 1);
-        if (lane == 0) before = m0;
-        const int t = t0 + lane;
-        // the token's own m from the m before it: the pair every consumer takes its weights from
+        if (lane == 0) before = start;
+        const int t = t0 + threadIdx.x;
+        // the token's own m beside the m before it: the pair every consumer takes its weights from
         if (t < hi) out[(size_t)t * heads + h] = make_float4(g.x, g.y, m, before);
-        m0 = __shfl_sync(0xffffffffu, m, min(31, hi - 1 - t0));
     }
-    if (write && lane == 0) *m_at = m0;
+    if (write && threadIdx.x == 0) *m_at = m0;
 }
 
 // c [tokens, channels] = silu(convolution) as the engine's type; unit [tokens, kv_heads] = factors that make q (times q_scale) and k unit
@@ -317,6 +327,95 @@ delta_prepare_kernel(const T* __restrict__ proj, int ld, const float* __restrict
         ssq = warp_sum(ssq);
         ssk = warp_sum(ssk);
         if (lane == 0) unit[(size_t)t * kv_heads + g] = make_float2(q_scale / sqrtf(ssq + tiny), 1.0f / sqrtf(ssk + tiny));
+    }
+}
+
+// The same for two channels a lane and taps known when compiling: a warp takes a run of tokens and one head of q, of k or of v (or, last,
+// the decays and step sizes of all heads), and the rows a run's convolutions share are read once.
+constexpr int kRun = 8;
+template <typename T> __device__ __forceinline__ float2 pair_of(const T* p);
+template <> __device__ __forceinline__ float2 pair_of<float>(const float* p) { return *reinterpret_cast<const float2*>(p); }
+template <> __device__ __forceinline__ float2 pair_of<bf16>(const bf16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+__device__ __forceinline__ float2 round_pair(float* p, float a, float b) {
+    *reinterpret_cast<float2*>(p) = make_float2(a, b);
+    return make_float2(a, b);
+}
+__device__ __forceinline__ float2 round_pair(bf16* p, float a, float b) {
+    const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+    *reinterpret_cast<__nv_bfloat162*>(p) = v;
+    return __bfloat1622float2(v);
+}
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128)
+delta_prepare_run_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ gates, const float* __restrict__ conv,
+                         const float* __restrict__ rate, const float* __restrict__ dt_bias, const float* __restrict__ state,
+                         long long slot_stride, long long ring_offset, const int* __restrict__ state_slots, const int* __restrict__ positions,
+                         const int* __restrict__ token_request, const int* __restrict__ cu_seqlens, T* __restrict__ c_out,
+                         float2* __restrict__ unit, float2* __restrict__ steps, int tokens, int heads, int kv_heads, int dim, int vdim,
+                         float tiny, float q_scale) {
+    pdl_trigger();
+    pdl_wait();
+    const int t0 = blockIdx.x * kRun, n = min(kRun, tokens - t0), lane = threadIdx.x & 31;
+    const int u = blockIdx.y * 4 + (threadIdx.x >> 5);
+    const int qk = kv_heads * dim, channels = 2 * qk + heads * vdim;
+    if (u > 2 * kv_heads + heads) return;
+    if (u == 2 * kv_heads + heads) {
+        for (int x = lane; x < n * heads; x += 32) {
+            const int h = x % heads;
+            const float* g = gates + (size_t)(t0 + x / heads) * 2 * heads;
+            steps[(size_t)t0 * heads + x] = make_float2(-rate[h] * soft_plus(g[heads + h] + dt_bias[h]), sigmoid_f(g[h]));
+        }
+        return;
+    }
+    const bool is_v = u >= 2 * kv_heads;
+    const int c0 = is_v ? 2 * qk + (u - 2 * kv_heads) * vdim : u * dim, width = is_v ? vdim : dim;
+    float ss[kRun];
+#pragma unroll
+    for (int r = 0; r < kRun; ++r) ss[r] = 0.f;
+    for (int i = 2 * lane; i < width; i += 64) {
+        const int c = c0 + i;
+        float w0[TAPS], w1[TAPS];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) { w0[j] = conv[(size_t)c * TAPS + j]; w1[j] = conv[(size_t)(c + 1) * TAPS + j]; }
+        float2 x[kRun];
+#pragma unroll
+        for (int r = 0; r < kRun; ++r)
+            if (r < n) x[r] = pair_of(proj + (size_t)(t0 + r) * ld + c);
+        float2 win[TAPS];              // the inputs of the current token's convolution, the oldest first
+        int b = -1;
+#pragma unroll
+        for (int r = 0; r < kRun; ++r) {
+            if (r >= n) continue;
+            const int t = t0 + r;
+            if (r == 0 || token_request[t] != b) {         // the run's start, or a request's first token of the step
+                b = token_request[t];
+                const int local = t - cu_seqlens[b], p = positions[t];
+                const float* ring = state + (size_t)state_slots[b] * slot_stride + ring_offset;
+#pragma unroll
+                for (int j = 0; j < TAPS - 1; ++j) {
+                    const int back = TAPS - 1 - j;
+                    win[j + 1] = back <= local ? pair_of(proj + (size_t)(t - back) * ld + c)
+                                               : make_float2(ring[(size_t)((p + 1 + j) % TAPS) * channels + c], ring[(size_t)((p + 1 + j) % TAPS) * channels + c + 1]);
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j) win[j] = win[j + 1];
+            win[TAPS - 1] = x[r];
+            float a0 = 0.f, a1 = 0.f;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) { a0 = fmaf(w0[j], win[j].x, a0); a1 = fmaf(w1[j], win[j].y, a1); }
+            const float2 y = round_pair(c_out + (size_t)t * channels + c, a0 * sigmoid_f(a0), a1 * sigmoid_f(a1));
+            ss[r] = fmaf(y.x, y.x, fmaf(y.y, y.y, ss[r]));
+        }
+    }
+    if (is_v) return;
+#pragma unroll
+    for (int r = 0; r < kRun; ++r) {
+        const float sum = warp_sum(ss[r]);
+        if (lane != 0 || r >= n) continue;
+        float* at = reinterpret_cast<float*>(unit + (size_t)(t0 + r) * kv_heads + u % kv_heads);
+        at[u / kv_heads] = (u < kv_heads ? q_scale : 1.0f) / sqrtf(sum + tiny);
     }
 }
 
@@ -492,6 +591,63 @@ state_finish_kernel(const float* __restrict__ o, int o_ld, const float4* __restr
     }
 }
 
+template <typename T> __device__ __forceinline__ float4 four_of(const T* p);
+template <> __device__ __forceinline__ float4 four_of<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <> __device__ __forceinline__ float4 four_of<bf16>(const bf16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void put_four(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put_four(bf16* p, float4 v) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+}
+
+// The same, four columns a lane and up to 128 * PER columns: everything a lane needs is asked for at once.
+template <typename T, int KIND, int PER>
+__global__ void __launch_bounds__(256)
+state_finish_vec_kernel(const float* __restrict__ o, int o_ld, const float4* __restrict__ gates, const T* __restrict__ proj, int ld, int z_col,
+                        const float* __restrict__ gain, T* __restrict__ out, int heads, int vdim, float eps, float tiny, long long rows) {
+    pdl_trigger();
+    pdl_wait();
+    const long long row = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (row >= rows) return;
+    const int lane = threadIdx.x & 31, h = (int)(row % heads);
+    const long long t = row / heads;
+    const float* x = o + row * o_ld;
+    const T* z_row = proj + (size_t)t * ld + z_col + h * vdim;
+    float4 v[PER], z[PER], g[PER];
+    float nq = 0.f, m = 0.f;
+    if (KIND == kMemory) { nq = x[vdim]; m = gates[row].z; }
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+        const int c = 4 * lane + 128 * j;
+        v[j] = z[j] = g[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < vdim) {
+            v[j] = four_of(x + c);
+            z[j] = four_of(z_row + c);
+            g[j] = four_of(gain + (KIND == kMemory ? h * vdim : 0) + c);
+        }
+    }
+    const float den = KIND == kMemory ? 1.0f / (fmaxf(fabsf(nq), expf(-m)) + tiny) : 1.0f;
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+        v[j] = make_float4(v[j].x * den, v[j].y * den, v[j].z * den, v[j].w * den);
+        ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + eps);
+    auto gate = [](float y) { const float sg = sigmoid_f(y); return KIND == kMemory ? sg : y * sg; };
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+        const int c = 4 * lane + 128 * j;
+        if (c < vdim)
+            put_four(out + (size_t)row * vdim + c, make_float4(v[j].x * inv * g[j].x * gate(z[j].x), v[j].y * inv * g[j].y * gate(z[j].y),
+                                                               v[j].z * inv * g[j].z * gate(z[j].z), v[j].w * inv * g[j].w * gate(z[j].w)));
+    }
+}
+
 // how a column's rows are shared out: lanes a column, four-number pieces a lane
 struct Split { int ds, pieces; };
 Split split_rows(int dim) {
@@ -582,7 +738,7 @@ LLM_API int llm_gated_delta_step(const void* proj, int ld, const float* gates, c
 LLM_API int llm_memory_gates(const float* gates, const float* bias, float cap, float* state, long long slot_stride, long long m_offset,
                              const int* state_slots, const int* cu_seqlens, void* out, int requests, int heads, int write, cudaStream_t stream) {
     if (requests == 0) return 0;
-    llm_launch(memory_gates_kernel, dim3((unsigned)requests, (unsigned)((heads + 3) / 4)), 128, 0, stream, gates, bias, cap, state, slot_stride,
+    llm_launch(memory_gates_kernel, dim3((unsigned)requests, (unsigned)heads), kGateThreads, 0, stream, gates, bias, cap, state, slot_stride,
                m_offset, state_slots, cu_seqlens, (float4*)out, heads, write);
     LLM_CHECK_LAUNCH("memory_gates");
     return 0;
@@ -601,11 +757,23 @@ LLM_API int llm_delta_prepare(const void* proj, int ld, const float* gates, cons
     const int channels = 2 * kv_heads * dim + heads * vdim;
     return llm_dispatch_dtype(dtype, [&](auto tag) {
         using T = decltype(tag);
+        const int units = 2 * kv_heads + heads + 1;
+        auto run = [&](auto kern) {
+            llm_launch(kern, dim3((unsigned)((tokens + kRun - 1) / kRun), (unsigned)((units + 3) / 4)), 128, 0, stream, (const T*)proj, ld, gates, conv,
+                       rate, dt_bias, (const float*)state, slot_stride, ring, state_slots, positions, token_request, cu_seqlens, (T*)c_out,
+                       (float2*)unit, (float2*)steps, tokens, heads, kv_heads, dim, vdim, tiny, q_scale);
+        };
         auto kern = delta_prepare_kernel<T>;
+        const bool pairs = dim % 2 == 0 && vdim % 2 == 0 && ld % 2 == 0;
+        if (pairs && taps == 2) run(delta_prepare_run_kernel<T, 2>);
+        else if (pairs && taps == 3) run(delta_prepare_run_kernel<T, 3>);
+        else if (pairs && taps == 4) run(delta_prepare_run_kernel<T, 4>);
+        else {
         if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         llm_launch(kern, (unsigned)tokens, 256, smem, stream, (const T*)proj, ld, gates, conv, rate, dt_bias, (const float*)state, slot_stride,
                    ring, state_slots, positions, token_request, cu_seqlens, (T*)c_out, (float2*)unit, (float2*)steps, heads, kv_heads, dim,
                    vdim, taps, tiny, q_scale);
+        }
         LLM_CHECK_LAUNCH("delta_prepare");
         if (write) {
             const int by = (channels + 255) / 256 < 16 ? (channels + 255) / 256 : 16;
@@ -638,7 +806,11 @@ LLM_API int llm_state_finish(int kind, const float* o, int o_ld, const void* gat
             llm_launch(kern, (unsigned)((rows + 7) / 8), 256, 0, stream, o, o_ld, (const float4*)gates, (const T*)proj, ld, z_col, gain, (T*)out, heads,
                        vdim, eps, tiny, rows);
         };
-        if (kind == kMemory) go(state_finish_kernel<T, kMemory>);
+        const bool fours = vdim % 4 == 0 && ld % 4 == 0 && z_col % 4 == 0 && o_ld % 4 == 0 && !((uintptr_t)proj & 15) && !((uintptr_t)out & 15) &&
+                           !((uintptr_t)gain & 15) && vdim <= 512;
+        if (fours && kind == kMemory) go(vdim <= 128 ? state_finish_vec_kernel<T, kMemory, 1> : state_finish_vec_kernel<T, kMemory, 4>);
+        else if (fours) go(vdim <= 128 ? state_finish_vec_kernel<T, kDelta, 1> : state_finish_vec_kernel<T, kDelta, 4>);
+        else if (kind == kMemory) go(state_finish_kernel<T, kMemory>);
         else go(state_finish_kernel<T, kDelta>);
         LLM_CHECK_LAUNCH("state_finish");
         return 0;
