@@ -39,7 +39,7 @@ def silu(z):
 
 
 def embedding(tokens, w, cfg):
-    return w["embed"][torch.tensor(tokens, dtype=torch.long)] * cfg["embedding"]["scale"]
+    return w["embed"][torch.tensor(tokens, dtype=torch.long)] * (cfg.get("embedding") or {"scale": 1.0})["scale"]
 
 
 # ---- mixer: matrix memory with exponential gates ------------------------------------------------------------------
@@ -80,6 +80,8 @@ def matrix_memory(h, w, p, m, eps):
 # ---- mixer: attention beside a gated delta rule -------------------------------------------------------------------
 def rotate_neighbours(x, dims, base):
     """x [T, n, D]: of the leading `dims` numbers of each row 2i rotates with 2i + 1, by position * base^(-2i/dims)."""
+    if not dims:
+        return x
     T = x.shape[0]
     f = torch.tensor([base ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64)
     a = torch.arange(T, dtype=torch.float64).view(T, 1, 1) * f.view(1, 1, -1)
@@ -97,7 +99,7 @@ def causal_softmax(s):
 
 def grouped_attention(h, w, p, m):
     T, H, G, D, V = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    rot = (int(m["rot"]["dims"]), float(m["rot"]["base"]))
+    rot = (int(m["rot"]["dims"]), float(m["rot"]["base"])) if m.get("rot") else (0, 1.0)
     q = rotate_neighbours((h @ w[p + "q"].T).view(T, H, D), *rot)
     k = rotate_neighbours((h @ w[p + "k"].T).view(T, G, D), *rot).repeat_interleave(H // G, dim=1)
     v = (h @ w[p + "v"].T).view(T, G, V).repeat_interleave(H // G, dim=1)
@@ -180,7 +182,7 @@ def experts(h, w, p, mlp):
 
 # ---- the model ----------------------------------------------------------------------------------------------------
 def layer(x, w, i, lay, cfg):
-    c, eps, p = cfg["residual_mult"], cfg["norm"]["eps"], f"l{i}."
+    c, eps, p = cfg.get("residual_mult", 1.0), cfg["norm"]["eps"], f"l{i}."
     x = x + c * MIXERS[lay["type"]](stream_norm(x, w, p + "norm1", eps), w, p + "mix.", lay["mixer"], eps)
     if lay["mlp"] is not None:
         h = stream_norm(x, w, p + "norm2", eps)

@@ -223,7 +223,7 @@ def test_add_branch_rmsnorm(K, dtype, T, width, form):
         close(delta.sum(), plain, dtype)
 
 
-@pytest.mark.parametrize("E,groups,top,scale", [(12, (3, 2), 4, 1.0), (8, (4, 1), 2, 2.5), (6, (6, 4), 3, 0.3), (40, (5, 5), 7, 1.2), (9, None, 2, 1.7)])
+@pytest.mark.parametrize("E,groups,top,scale", [(15, (3, 2), 5, 1.0), (8, (4, 1), 2, 2.5), (6, (6, 4), 3, 0.3), (40, (5, 5), 7, 1.2), (9, None, 2, 1.7)])
 def test_route_topk_two_best_of_a_group(K, E, groups, top, scale):
     z = rnd(33, E, seed=E)
     chosen, weights = torch.empty(33, top, dtype=torch.int32, device="cuda"), torch.empty(33, top, device="cuda")
