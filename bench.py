@@ -153,7 +153,7 @@ def main() -> int:
     ap.add_argument("--family", choices=["lifusun", "rodapel", "fomerax", "mamusun", "bidinex", "kobolix"], default=None,
                     help="instead of the headline line: prefill and decode of this family at the layer sizes of --shape "
                          "(8b, 3b, 1b, toy; eight layers) beside a Llama of the same sizes and depth (fomerax and mamusun: also beside the "
-                         "Rodapel of those sizes), and its kernels alone")
+                         "Rodapel of those sizes, bidinex: the Fomerax, kobolix: the Mamusun), and its kernels alone")
     args = ap.parse_args()
     if args.family:
         from iitj_llm_coopt_b200.family_bench import run as family_run

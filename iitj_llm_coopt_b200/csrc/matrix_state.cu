@@ -347,7 +347,7 @@ __device__ __forceinline__ float2 round_pair(bf16* p, float a, float b) {
 }
 
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, 8)
 delta_prepare_run_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ gates, const float* __restrict__ conv,
                          const float* __restrict__ rate, const float* __restrict__ dt_bias, const float* __restrict__ state,
                          long long slot_stride, long long ring_offset, const int* __restrict__ state_slots, const int* __restrict__ positions,
@@ -375,9 +375,13 @@ delta_prepare_run_kernel(const T* __restrict__ proj, int ld, const float* __rest
     for (int r = 0; r < kRun; ++r) ss[r] = 0.f;
     for (int i = 2 * lane; i < width; i += 64) {
         const int c = c0 + i;
-        float w0[TAPS], w1[TAPS];
+        float w[2 * TAPS];             // both channels' taps lie side by side
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) { w0[j] = conv[(size_t)c * TAPS + j]; w1[j] = conv[(size_t)(c + 1) * TAPS + j]; }
+        for (int j = 0; j < TAPS; ++j) {
+            const float2 v = *reinterpret_cast<const float2*>(conv + (size_t)c * TAPS + 2 * j);
+            w[2 * j] = v.x;
+            w[2 * j + 1] = v.y;
+        }
         float2 x[kRun];
 #pragma unroll
         for (int r = 0; r < kRun; ++r)
@@ -404,7 +408,7 @@ delta_prepare_run_kernel(const T* __restrict__ proj, int ld, const float* __rest
             win[TAPS - 1] = x[r];
             float a0 = 0.f, a1 = 0.f;
 #pragma unroll
-            for (int j = 0; j < TAPS; ++j) { a0 = fmaf(w0[j], win[j].x, a0); a1 = fmaf(w1[j], win[j].y, a1); }
+            for (int j = 0; j < TAPS; ++j) { a0 = fmaf(w[j], win[j].x, a0); a1 = fmaf(w[TAPS + j], win[j].y, a1); }
             const float2 y = round_pair(c_out + (size_t)t * channels + c, a0 * sigmoid_f(a0), a1 * sigmoid_f(a1));
             ss[r] = fmaf(y.x, y.x, fmaf(y.y, y.y, ss[r]));
         }
@@ -764,7 +768,7 @@ LLM_API int llm_delta_prepare(const void* proj, int ld, const float* gates, cons
                        (float2*)unit, (float2*)steps, tokens, heads, kv_heads, dim, vdim, tiny, q_scale);
         };
         auto kern = delta_prepare_kernel<T>;
-        const bool pairs = dim % 2 == 0 && vdim % 2 == 0 && ld % 2 == 0;
+        const bool pairs = dim % 2 == 0 && vdim % 2 == 0 && ld % 2 == 0 && !((uintptr_t)conv & 7);
         if (pairs && taps == 2) run(delta_prepare_run_kernel<T, 2>);
         else if (pairs && taps == 3) run(delta_prepare_run_kernel<T, 3>);
         else if (pairs && taps == 4) run(delta_prepare_run_kernel<T, 4>);

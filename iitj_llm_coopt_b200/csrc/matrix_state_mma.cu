@@ -281,11 +281,12 @@ memory_out_kernel(MemoryArgs a) {
         }
     }
     const int t[2] = {row + (lane >> 2), row + (lane >> 2) + 8};
-    float norm[2] = {0.f, 0.f}, e[2], fm[2];
+    float norm[2] = {0.f, 0.f}, e[2], ft[2], mt[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
-        fm[r] = F[t[r]] - M[t[r]];
-        e[r] = t[r] < ch.z ? expf(fm[r] + m0) : 0.f;
+        ft[r] = F[t[r]];
+        mt[r] = M[t[r]];
+        e[r] = t[r] < ch.z ? expf(ft[r] + (m0 - mt[r])) : 0.f;
     }
 #pragma unroll
     for (int n = 0; n < 8; ++n)
@@ -301,7 +302,7 @@ memory_out_kernel(MemoryArgs a) {
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
                 const int key = n * 16 + half * 8 + 2 * (lane & 3) + (x & 1), r = x >> 1;
-                p[x] = key <= t[r] && t[r] < ch.z ? p[x] * expf(fm[r] + (I[key] - F[key])) : 0.f;
+                p[x] = key <= t[r] && t[r] < ch.z ? p[x] * expf((ft[r] - F[key]) + (I[key] - mt[r])) : 0.f;     // near keys first: long sums cancel
                 norm[r] += p[x];
             }
             split2(p[0], p[1], hi[2 * half], lo[2 * half]);
