@@ -575,13 +575,13 @@ state_walk_kernel(WalkArgs a) {
 template <typename T, int KIND>
 __global__ void __launch_bounds__(256)
 state_finish_kernel(const float* __restrict__ o, int o_ld, const float4* __restrict__ gates, const T* __restrict__ proj, int ld, int z_col,
-                    const float* __restrict__ gain, T* __restrict__ out, int heads, int vdim, float eps, float tiny, long long rows) {
+                    const float* __restrict__ gain, T* __restrict__ out, int heads, int vdim, float eps, float tiny, unsigned rows) {
     pdl_trigger();
     pdl_wait();
-    const long long row = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
-    if (row >= rows) return;
-    const int lane = threadIdx.x & 31, h = (int)(row % heads);
-    const long long t = row / heads;
+    const unsigned index = blockIdx.x * 8 + (threadIdx.x >> 5), token = index / (unsigned)heads;      // (the launcher keeps them in 32 bits)
+    if (index >= rows) return;
+    const int lane = threadIdx.x & 31, h = (int)(index - token * (unsigned)heads);
+    const size_t row = index, t = token;
     const float* x = o + row * o_ld;
     float den = 1.f;
     if (KIND == kMemory) den = 1.0f / (fmaxf(fabsf(x[vdim]), expf(-gates[row].z)) + tiny);
@@ -612,13 +612,13 @@ __device__ __forceinline__ void put_four(bf16* p, float4 v) {
 template <typename T, int KIND, int PER>
 __global__ void __launch_bounds__(256)
 state_finish_vec_kernel(const float* __restrict__ o, int o_ld, const float4* __restrict__ gates, const T* __restrict__ proj, int ld, int z_col,
-                        const float* __restrict__ gain, T* __restrict__ out, int heads, int vdim, float eps, float tiny, long long rows) {
+                        const float* __restrict__ gain, T* __restrict__ out, int heads, int vdim, float eps, float tiny, unsigned rows) {
     pdl_trigger();
     pdl_wait();
-    const long long row = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
-    if (row >= rows) return;
-    const int lane = threadIdx.x & 31, h = (int)(row % heads);
-    const long long t = row / heads;
+    const unsigned index = blockIdx.x * 8 + (threadIdx.x >> 5), token = index / (unsigned)heads;      // (the launcher keeps them in 32 bits)
+    if (index >= rows) return;
+    const int lane = threadIdx.x & 31, h = (int)(index - token * (unsigned)heads);
+    const size_t row = index, t = token;
     const float* x = o + row * o_ld;
     const T* z_row = proj + (size_t)t * ld + z_col + h * vdim;
     float4 v[PER], z[PER], g[PER];
@@ -804,11 +804,12 @@ LLM_API int llm_state_finish(int kind, const float* o, int o_ld, const void* gat
                              int dtype, int tokens, int heads, int vdim, float eps, float tiny, cudaStream_t stream) {
     if (tokens == 0) return 0;
     const long long rows = (long long)tokens * heads;
+    if (rows > 0x7ffffff0LL) LLM_FAIL(-1, "state_finish: %d tokens of %d heads are too many for a launch", tokens, heads);
     return llm_dispatch_dtype(dtype, [&](auto tag) {
         using T = decltype(tag);
         auto go = [&](auto kern) {
             llm_launch(kern, (unsigned)((rows + 7) / 8), 256, 0, stream, o, o_ld, (const float4*)gates, (const T*)proj, ld, z_col, gain, (T*)out, heads,
-                       vdim, eps, tiny, rows);
+                       vdim, eps, tiny, (unsigned)rows);
         };
         const bool fours = vdim % 4 == 0 && ld % 4 == 0 && z_col % 4 == 0 && o_ld % 4 == 0 && !((uintptr_t)proj & 15) && !((uintptr_t)out & 15) &&
                            !((uintptr_t)gain & 15) && vdim <= 512;
